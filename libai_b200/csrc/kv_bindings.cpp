@@ -37,15 +37,16 @@ int lbk_ring_decode(const void* q, long ldq, const void* ring, const void* first
                     const void* gate, long ldg, void* y, long ldy, float* part, int B, int H, int G, int D, int V, int window,
                     int chunk, int keep, float scale, int splits, float softcap, int sink, int gate_wide, float out_scale, int dtype,
                     cudaStream_t s);
-int lbk_moe_topk(const float* z, long ldz, const float* bias, int mode, int E, int top, float rscale, int* idx, float* wts, int* counts,
-                 long tokens, cudaStream_t s);
+int lbk_moe_topk(const float* z, long ldz, const float* bias, const float* corr, int mode, int E, int real, int top, float rscale, int* idx,
+                 float* wts, int* counts, float* keep, long tokens, cudaStream_t s);
 int lbk_moe_pairs(const void* h, long ldh, const void* wgu, const void* wd, const int* idx, const float* wts, void* a, float* out,
-                  long tokens, int ff, int n, int top, int act, float limit, int win, int dtype, cudaStream_t s);
+                  long tokens, int E, int ff, int n, int top, int act, int gated, float limit, int win, int dtype, cudaStream_t s);
 int lbk_moe_sort(const void* h, long ldh, const int* idx, const int* counts, int* offsets, int* cursor, int* pos, void* xs, long tokens,
                  int E, int n, int top, int align, int* tile_group, int tiles, const float* wts, int dtype, cudaStream_t s);
 int lbp_postnorm_residual(const float* xin, float* xout, const void* y1, long ldy1, int y1dtype, const float* y2, long ldy2,
-                          const int* pos, const float* cw, int top, float alpha, const void* w, float eps, void* h, long ldh,
-                          long rows, int n, int dtype, cudaStream_t s);
+                          const int* pos, const float* cw, int top, float alpha, const float* gate, long ldgate, const float* keep,
+                          int outer, float out_scale, const void* w, float eps, void* h, long ldh, long rows, int n, int dtype,
+                          cudaStream_t s);
 int lbp_conv_qkv_prepare(const void* qin, const void* kin, const void* vin, long ld, const void* wq, const void* wk, const void* wv,
                          int taps, void* tail, const void* qn, const void* kn, const float* freq, int half, float eps, void* qout,
                          long ldqo, void* pool, const int* table, int max_pages, int page_size, const int* tok_seq,
@@ -251,34 +252,43 @@ void ring_attention(const Tensor& q, const Tensor& ring, const Tensor& first, co
         "ring_attention");
 }
 
-void moe_topk(const Tensor& z, const OptT& bias, int64_t mode, int64_t top, double rscale, Tensor idx, Tensor wts, const OptT& counts) {
+// E: how many leading columns of z are choices (-1: all); the first `real` of them are experts, the rest identity experts
+void moe_topk(const Tensor& z, const OptT& bias, int64_t mode, int64_t top, double rscale, Tensor idx, Tensor wts, const OptT& counts,
+              const OptT& corr, int64_t E, int64_t real, const OptT& keep) {
+  if (E < 0) E = z.size(1);
+  if (real < 0) real = E;
+  TORCH_CHECK(E >= 1 && E <= z.size(1) && real >= 1 && real <= E && top >= 1 && top <= E, "moe_topk: choices, experts and top");
   rows2d(z, "moe_topk z");
   TORCH_CHECK(z.scalar_type() == at::kFloat, "moe_topk: fp32 router logits expected");
   TORCH_CHECK(idx.is_cuda() && idx.scalar_type() == at::kInt && idx.is_contiguous() && idx.numel() == z.size(0) * top, "moe_topk: idx int32 [tokens, top]");
   TORCH_CHECK(wts.is_cuda() && wts.scalar_type() == at::kFloat && wts.is_contiguous() && wts.numel() == z.size(0) * top, "moe_topk: weights fp32 [tokens, top]");
   const float* bp = nullptr;
-  if (has(bias)) { TORCH_CHECK(bias->is_cuda() && bias->scalar_type() == at::kFloat && bias->is_contiguous() && bias->numel() == z.size(1), "moe_topk: bias fp32 [E]"); bp = bias->data_ptr<float>(); }
-  TORCH_CHECK(mode >= 0 && mode <= 2, "moe_topk: mode 0 (sigmoid scores, normalised), 1 (softmax over the chosen logits) or 2 (sigmoid scores as they are)");
+  if (has(bias)) { TORCH_CHECK(bias->is_cuda() && bias->scalar_type() == at::kFloat && bias->is_contiguous() && bias->numel() == E, "moe_topk: bias fp32 [E]"); bp = bias->data_ptr<float>(); }
+  TORCH_CHECK(mode >= 0 && mode <= 3, "moe_topk: mode 0 (sigmoid scores, normalised), 1 (softmax over the chosen logits), 2 (sigmoid scores as they are) or 3 (softmax scores over all choices as they are)");
+  const float* cr = nullptr; float* kp = nullptr;
+  if (has(corr)) { TORCH_CHECK(mode == 3 && corr->is_cuda() && corr->scalar_type() == at::kFloat && corr->is_contiguous() && corr->numel() == E, "moe_topk: correction fp32 [E] (mode 3)"); cr = corr->data_ptr<float>(); }
+  if (has(keep)) { TORCH_CHECK(keep->is_cuda() && keep->scalar_type() == at::kFloat && keep->is_contiguous() && keep->numel() == z.size(0), "moe_topk: keep fp32 [tokens]"); kp = keep->data_ptr<float>(); }
   int* cp = nullptr;
-  if (has(counts)) { TORCH_CHECK(counts->is_cuda() && counts->scalar_type() == at::kInt && counts->numel() >= z.size(1), "moe_topk: counts"); cp = counts->data_ptr<int>(); }
+  if (has(counts)) { TORCH_CHECK(counts->is_cuda() && counts->scalar_type() == at::kInt && counts->numel() >= real, "moe_topk: counts"); cp = counts->data_ptr<int>(); }
   c10::cuda::CUDAGuard guard(z.device());
-  check(lbk_moe_topk(z.data_ptr<float>(), z.stride(0), bp, (int)mode, (int)z.size(1), (int)top, (float)rscale, idx.data_ptr<int>(), wts.data_ptr<float>(), cp,
-                     z.size(0), cur_stream()), "moe_topk");
+  check(lbk_moe_topk(z.data_ptr<float>(), z.stride(0), bp, cr, (int)mode, (int)E, (int)real, (int)top, (float)rscale, idx.data_ptr<int>(),
+                     wts.data_ptr<float>(), cp, kp, z.size(0), cur_stream()), "moe_topk");
 }
 
 void moe_pairs(const Tensor& h, const Tensor& wgu, const Tensor& wd, const Tensor& idx, const Tensor& wts, Tensor a, Tensor out, int64_t act,
-               double limit, bool weight_input) {
+               double limit, bool weight_input, bool gated) {
   rows2d(h, "moe_pairs h");
   const int64_t n = h.size(1), tokens = h.size(0), top = idx.numel() / std::max<int64_t>(tokens, 1);
-  TORCH_CHECK(wgu.is_cuda() && wgu.dim() == 3 && wgu.is_contiguous() && wgu.size(2) == n && wgu.size(1) % 2 == 0 && code(wgu) == code(h), "moe_pairs: wgu [E, 2 ff, width]");
-  const int64_t ff = wgu.size(1) / 2;
+  TORCH_CHECK(wgu.is_cuda() && wgu.dim() == 3 && wgu.is_contiguous() && wgu.size(2) == n && (!gated || wgu.size(1) % 2 == 0) && code(wgu) == code(h), "moe_pairs: wgu [E, 2 ff (ff without a gate), width]");
+  const int64_t ff = gated ? wgu.size(1) / 2 : wgu.size(1);
   TORCH_CHECK(wd.is_cuda() && wd.dim() == 3 && wd.is_contiguous() && wd.size(0) == wgu.size(0) && wd.size(1) == n && wd.size(2) == ff && code(wd) == code(h), "moe_pairs: wd [E, width, ff]");
   TORCH_CHECK(a.is_cuda() && a.is_contiguous() && a.numel() == tokens * top * ff && code(a) == code(h), "moe_pairs: a [tokens*top, ff]");
   TORCH_CHECK(out.is_cuda() && out.scalar_type() == at::kFloat && out.is_contiguous() && out.numel() == tokens * n, "moe_pairs: out fp32 [tokens, width]");
   TORCH_CHECK(wts.scalar_type() == at::kFloat && wts.is_contiguous() && wts.numel() == idx.numel(), "moe_pairs: weights");
   c10::cuda::CUDAGuard guard(h.device());
   check(lbk_moe_pairs(h.data_ptr(), h.stride(0), wgu.data_ptr(), wd.data_ptr(), meta(idx), wts.data_ptr<float>(), a.data_ptr(), out.data_ptr<float>(),
-                      tokens, (int)ff, (int)n, (int)top, (int)act, (float)limit, weight_input ? 1 : 0, code(h), cur_stream()), "moe_pairs");
+                      tokens, (int)wgu.size(0), (int)ff, (int)n, (int)top, (int)act, gated ? 1 : 0, (float)limit, weight_input ? 1 : 0, code(h), cur_stream()),
+        "moe_pairs");
 }
 
 // rows sorted by expert; with `tile_group` (int32 [rows of xs / align]) every expert's range starts on a multiple of `align`
@@ -305,9 +315,10 @@ void moe_sort(const Tensor& h, const Tensor& idx, const Tensor& counts, Tensor o
         "moe_sort");
 }
 
-// x fp32 [rows, n]: out = rmsnorm(alpha x + y1 + y2') (1 + w) into xout (fp32, may be x) and h (the model's dtype)
+// x fp32 [rows, n]: v = (alpha + keep[r]) x + sigmoid(gate[r]) y1 + y2', o = rmsnorm(v) (1 + w) * out_scale; o — or, with `outer`, x + o —
+// goes into xout (fp32, may be x) and h (the model's dtype).  gate: fp32 [rows] or a column of an fp32 matrix
 void postnorm_residual(const Tensor& x, const OptT& xout, const OptT& y1, const OptT& y2, const OptT& pos, const OptT& cw, double alpha,
-                       const Tensor& w, double eps, const OptT& h) {
+                       const Tensor& w, double eps, const OptT& h, const OptT& gate, const OptT& keep, bool outer, double out_scale) {
   TORCH_CHECK(x.is_cuda() && x.dim() == 2 && x.is_contiguous() && x.scalar_type() == at::kFloat, "postnorm_residual: x fp32 [rows, width]");
   const int64_t rows = x.size(0), n = x.size(1);
   const int dtype = code(w);
@@ -339,6 +350,15 @@ void postnorm_residual(const Tensor& x, const OptT& xout, const OptT& y1, const 
       TORCH_CHECK(y2->size(0) == rows, "postnorm_residual: y2 rows");
     }
   }
+  const float* gp = nullptr; long ldgate = 0; const float* kp = nullptr;
+  if (has(gate)) {
+    TORCH_CHECK(y1p && gate->is_cuda() && gate->scalar_type() == at::kFloat && gate->dim() == 1 && gate->size(0) == rows, "postnorm_residual: gate fp32 [rows] (scales y1)");
+    gp = gate->data_ptr<float>(); ldgate = gate->stride(0);
+  }
+  if (has(keep)) {
+    TORCH_CHECK(keep->is_cuda() && keep->scalar_type() == at::kFloat && keep->is_contiguous() && keep->numel() == rows, "postnorm_residual: keep fp32 [rows]");
+    kp = keep->data_ptr<float>();
+  }
   void* hp = nullptr; long ldh = 0;
   if (has(h)) {
     rows2d(*h, "postnorm_residual h");
@@ -346,8 +366,8 @@ void postnorm_residual(const Tensor& x, const OptT& xout, const OptT& y1, const 
     hp = h->data_ptr(); ldh = h->stride(0);
   }
   c10::cuda::CUDAGuard guard(x.device());
-  check(lbp_postnorm_residual(x.data_ptr<float>(), xo, y1p, ldy1, y1d, y2p, ldy2, pp, cp, top, (float)alpha, w.data_ptr(), (float)eps, hp, ldh,
-                              rows, (int)n, dtype, cur_stream()), "postnorm_residual");
+  check(lbp_postnorm_residual(x.data_ptr<float>(), xo, y1p, ldy1, y1d, y2p, ldy2, pp, cp, top, (float)alpha, gp, ldgate, kp,
+                              outer ? 1 : 0, (float)out_scale, w.data_ptr(), (float)eps, hp, ldh, rows, (int)n, dtype, cur_stream()), "postnorm_residual");
 }
 
 // q, k, v: column slices of one projection output (one row stride).  tail [slots, taps-1, H*D + G*D + G*V]; pool
@@ -430,10 +450,10 @@ TORCH_LIBRARY(libai_b200_kv, m) {
   m.def("kv_gather(Tensor ring, Tensor first, Tensor knew, Tensor vnew, Tensor ext_seq, Tensor ext_off, Tensor nsink, Tensor cstart, Tensor seq_off, Tensor slots, Tensor past, Tensor(a!) ext) -> ()", &kv_gather);
   m.def("masked_attention(Tensor q, Tensor kmat, Tensor vmat, Tensor ext_off, Tensor nsink, Tensor cstart, Tensor? gate, Tensor tok_seq, Tensor seq_off, Tensor past, Tensor? qt_seq, Tensor? qt_start, Tensor(a!) y, int H, int G, int D, int V, int window, int chunk, int keep, float scale, float softcap=0.0, bool sink=False, bool gate_wide=False, float out_scale=1.0) -> ()", &masked_attention);
   m.def("ring_attention(Tensor q, Tensor ring, Tensor first, Tensor? gate, Tensor tok_seq, Tensor seq_off, Tensor slots, Tensor past, Tensor(a!) y, int H, int G, int D, int V, int window, int chunk, int keep, float scale, int splits, float softcap=0.0, bool sink=False, bool gate_wide=False, float out_scale=1.0) -> ()", &ring_attention);
-  m.def("moe_topk(Tensor z, Tensor? bias, int mode, int top, float rscale, Tensor(a!) idx, Tensor(b!) wts, Tensor(c!)? counts) -> ()", &moe_topk);
-  m.def("moe_pairs(Tensor h, Tensor wgu, Tensor wd, Tensor idx, Tensor wts, Tensor(a!) a, Tensor(b!) out, int act, float limit=0.0, bool weight_input=False) -> ()", &moe_pairs);
+  m.def("moe_topk(Tensor z, Tensor? bias, int mode, int top, float rscale, Tensor(a!) idx, Tensor(b!) wts, Tensor(c!)? counts, Tensor? corr=None, int E=-1, int real=-1, Tensor(d!)? keep=None) -> ()", &moe_topk);
+  m.def("moe_pairs(Tensor h, Tensor wgu, Tensor wd, Tensor idx, Tensor wts, Tensor(a!) a, Tensor(b!) out, int act, float limit=0.0, bool weight_input=False, bool gated=True) -> ()", &moe_pairs);
   m.def("moe_sort(Tensor h, Tensor idx, Tensor counts, Tensor(a!) offsets, Tensor(b!) cursor, Tensor(c!) pos, Tensor(d!) xs, int align, Tensor(e!)? tile_group, Tensor? wts=None) -> ()", &moe_sort);
-  m.def("postnorm_residual(Tensor x, Tensor(a!)? xout, Tensor? y1, Tensor? y2, Tensor? pos, Tensor? cw, float alpha, Tensor w, float eps, Tensor(b!)? h) -> ()", &postnorm_residual);
+  m.def("postnorm_residual(Tensor x, Tensor(a!)? xout, Tensor? y1, Tensor? y2, Tensor? pos, Tensor? cw, float alpha, Tensor w, float eps, Tensor(b!)? h, Tensor? gate=None, Tensor? keep=None, bool outer=False, float out_scale=1.0) -> ()", &postnorm_residual);
   m.def("conv_qkv_prepare(Tensor q, Tensor k, Tensor v, Tensor wq, Tensor wk, Tensor wv, Tensor(a!) tail, Tensor qn, Tensor kn, Tensor freq, float eps, Tensor(b!) qout, Tensor(c!) pool, Tensor table, Tensor tok_seq, Tensor seq_off, Tensor slots, Tensor past, int H, int G, int D, int V) -> ()", &conv_qkv_prepare);
   m.def("talk_attention_tiles(int qt_max, int H, int G, int D, int V) -> int[]", &talk_attention_tiles);
   m.def("talk_attention(Tensor q, Tensor pool, Tensor table, Tensor? talk, Tensor? sink, Tensor qt_seq, Tensor? qt_start, int QT, int KT, Tensor seq_off, Tensor slots, Tensor past, Tensor(a!) y, Tensor(b!)? part, int nparts, int H, int G, int D, int V, float scale, float out_scale) -> ()", &talk_attention);

@@ -882,27 +882,42 @@ __global__ void ring_decode_merge_kernel(const float* __restrict__ part, const T
 // Mixture of experts.
 //   moe_topk    : from the fp32 router logits z = W_r h (a product of the caller's): s = sigmoid(z), the `top` largest
 //                 (ties: the lower index), weights s / (sum + 1e-20) * rscale (mode 2: the scores themselves, s * rscale);
-//                 optionally counts the tokens of every expert.
+//                 mode 3: s = softmax(z) over all choices, the `top` largest s + corr, weights s * rscale; optionally counts
+//                 the tokens of every expert.  Choices at or above `real` are identity experts (their output is the token's
+//                 own input): they are never counted and the sum of their weights goes to `keep`.
 //   pair kernels: few tokens (single-token steps): every (token, chosen expert) pair reads its expert's matrices —
 //                 a = act(W_gate h) * (W_up h), then out[t] = sum_k weight_k W_down,k a_k in fp32.  `win` puts the weight on
 //                 the expert's input instead: the pair reads weight_k * h (rounded to T) and the outputs are summed.
 //   sort kernels: many tokens: rows are copied into a matrix sorted by expert (offsets from the counts), the experts
 //                 run as dense products on their row ranges, and the fused residual kernel gathers the weighted sum.
-// Expert matrices are stacked: wgu [E, 2*ff, n] (gate rows, then up rows), wd [E, n, ff].
+// Expert matrices are stacked: wgu [E, 2*ff, n] (gate rows, then up rows; [E, ff, n] without a gate), wd [E, n, ff].  A pair
+// whose expert number is E or more belongs to an identity expert: the pair kernels skip it, the sort gives it row -1.
 // ------------------------------------------------------------------------------------------------------------------
 // one warp per token over its fp32 router logits z [tokens, E] (+ bias [E] when given).  mode 0: scores sigmoid(z), weights
 // score / (sum of the chosen scores + 1e-20) * rscale; mode 1: scores z, weights = softmax over the chosen logits, times rscale;
-// mode 2: scores sigmoid(z), weights = the chosen scores as they are, times rscale
-__global__ void moe_topk_kernel(const float* __restrict__ z, long ldz, const float* __restrict__ bias, int mode, int E, int top,
-                                float rscale, int* __restrict__ idx, float* __restrict__ wts, int* __restrict__ counts, long tokens) {
+// mode 2: scores sigmoid(z), weights = the chosen scores as they are, times rscale; mode 3: scores softmax(z) over all E, chosen
+// by score + corr, weights = the chosen scores as they are, times rscale
+__global__ void moe_topk_kernel(const float* __restrict__ z, long ldz, const float* __restrict__ bias, const float* __restrict__ corr,
+                                int mode, int E, int real, int top, float rscale, int* __restrict__ idx, float* __restrict__ wts,
+                                int* __restrict__ counts, float* __restrict__ keep, long tokens) {
   extern __shared__ float sm[];
   const int wib = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const long tok = (long)blockIdx.x * nw + wib;
   float* sc = sm + (long)wib * E;
+  float* ws = sm + (long)(nw + wib) * E;         // mode 3: the scores without the correction
   if (tok >= tokens) return;                     // warps are independent below
+  float zmax = -INFINITY;
   for (int e = lane; e < E; e += 32) {
     const float v = z[tok * ldz + e] + (bias ? bias[e] : 0.f);
-    sc[e] = mode == 1 ? v : sigmoidf_(v);
+    sc[e] = (mode & 1) ? v : sigmoidf_(v);
+    zmax = fmaxf(zmax, v);
+  }
+  if (mode == 3) {
+    zmax = warp_max(zmax);
+    float zs = 0.f;
+    for (int e = lane; e < E; e += 32) { const float v = expf(sc[e] - zmax); ws[e] = v; zs += v; }
+    zs = warp_sum(zs);
+    for (int e = lane; e < E; e += 32) { const float v = ws[e] / zs; ws[e] = v; sc[e] = v + (corr ? corr[e] : 0.f); }
   }
   __syncwarp();
   float sum = 0.f, mine_w = 0.f, first = 0.f; int mine_e = 0;
@@ -915,8 +930,9 @@ __global__ void moe_topk_kernel(const float* __restrict__ z, long ldz, const flo
       const int oe = __shfl_xor_sync(0xffffffffu, be, mk);
       if (ov > best || (ov == best && oe < be)) { best = ov; be = oe; }
     }
+    if (be >= E) be = 0;                         // only when no score compares (NaN): the index stays in range
     if (k == 0) first = best;
-    const float wk = mode != 1 ? best : expf(best - first);   // the first choice is the largest logit
+    const float wk = mode == 3 ? ws[be] : (mode != 1 ? best : expf(best - first));   // mode 1: the first choice is the largest logit
     sum += wk;
     if (lane == k % 32) { mine_w = wk; mine_e = be; }
     if (lane == 0) sc[be] = -INFINITY;
@@ -927,21 +943,28 @@ __global__ void moe_topk_kernel(const float* __restrict__ z, long ldz, const flo
     }
   }
   __syncwarp();
-  const float inv = mode == 2 ? rscale : rscale / (mode == 0 ? sum + 1e-20f : sum);
+  const float inv = mode >= 2 ? rscale : rscale / (mode == 0 ? sum + 1e-20f : sum);
+  float own = 0.f;
   for (int k = lane; k < top; k += 32) {
-    wts[tok * top + k] *= inv;
-    if (counts) atomicAdd(counts + idx[tok * top + k], 1);
+    const float wk = wts[tok * top + k] * inv;
+    const int e = idx[tok * top + k];
+    wts[tok * top + k] = wk;
+    if (e >= real) own += wk;
+    else if (counts) atomicAdd(counts + e, 1);
   }
+  if (keep) { own = warp_sum(own); if (lane == 0) keep[tok] = own; }
 }
 
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_pair_gateup_kernel(const T* __restrict__ h, long ldh, const T* __restrict__ wgu, const int* __restrict__ idx,
-                       const float* __restrict__ wts, int win, T* __restrict__ a, int ff, int n, int top, int act, float limit) {
+                       const float* __restrict__ wts, int win, T* __restrict__ a, int E, int ff, int n, int top, int act, int gated,
+                       float limit) {
   extern __shared__ float sm[];
   const long pair = blockIdx.x;
   const long tok = pair / top;
   const int e = idx[pair];
+  if (e >= E) return;                            // an identity expert: the whole block leaves
   if (win) {
     const float wp = wts[pair];
     for (int i = threadIdx.x; i < n; i += blockDim.x) { T r; stf(&r, wp * ldf(h + tok * ldh + i)); sm[i] = ldf(&r); }
@@ -952,8 +975,13 @@ moe_pair_gateup_kernel(const T* __restrict__ h, long ldh, const T* __restrict__ 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int per = (ff + gridDim.y - 1) / gridDim.y;
   const int f0 = blockIdx.y * per, f1 = min(ff, f0 + per);
-  const T* wg = wgu + (long)e * 2 * ff * n;
+  const T* wg = wgu + (long)e * (gated ? 2 : 1) * ff * n;
   for (int f = f0 + warp; f < f1; f += nw) {
+    if (!gated) {
+      const float v = warp_dot<T>(wg + (long)f * n, sm, n, lane);
+      if (lane == 0) stf(a + pair * ff + f, act_apply(v, act));
+      continue;
+    }
     const float gv = warp_dot<T>(wg + (long)f * n, sm, n, lane);
     const float uv = warp_dot<T>(wg + (long)(ff + f) * n, sm, n, lane);
     if (lane == 0) stf(a + pair * ff + f, gated_apply(gv, uv, act, limit));
@@ -963,10 +991,10 @@ moe_pair_gateup_kernel(const T* __restrict__ h, long ldh, const T* __restrict__ 
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_pair_down_kernel(const T* __restrict__ a, const T* __restrict__ wd, const int* __restrict__ idx, const float* __restrict__ wts,
-                     int win, float* __restrict__ out, int ff, int n, int top) {
+                     int win, float* __restrict__ out, int E, int ff, int n, int top) {
   extern __shared__ float sm[];
   const long tok = blockIdx.x;
-  for (int i = threadIdx.x; i < top * ff; i += blockDim.x) sm[i] = ldf(a + tok * top * ff + i);
+  for (int i = threadIdx.x; i < top * ff; i += blockDim.x) if (idx[tok * top + i / ff] < E) sm[i] = ldf(a + tok * top * ff + i);
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int per = (n + gridDim.y - 1) / gridDim.y;
@@ -975,6 +1003,7 @@ moe_pair_down_kernel(const T* __restrict__ a, const T* __restrict__ wd, const in
     float acc = 0.f;
     for (int k = 0; k < top; ++k) {
       const int e = idx[tok * top + k];
+      if (e >= E) continue;
       acc += (win ? 1.f : wts[tok * top + k]) * warp_dot<T>(wd + ((long)e * n + c) * ff, sm + k * ff, ff, lane);
     }
     if (lane == 0) out[tok * n + c] = acc;
@@ -1008,16 +1037,17 @@ __global__ void moe_offsets_kernel(const int* __restrict__ counts, int* __restri
 
 template <typename T>
 __global__ void moe_scatter_kernel(const T* __restrict__ h, long ldh, const int* __restrict__ idx, const int* __restrict__ offsets,
-                                   int* __restrict__ cursor, int* __restrict__ pos, T* __restrict__ xs, int n, int top,
+                                   int* __restrict__ cursor, int* __restrict__ pos, T* __restrict__ xs, int E, int n, int top,
                                    const float* __restrict__ wts) {   // wts given: the copied row is wts[pair] * h
   __shared__ int where;
   const long pair = blockIdx.x;
   if (threadIdx.x == 0) {
     const int e = idx[pair];
-    where = offsets[e] + atomicAdd(cursor + e, 1);
+    where = e < E ? offsets[e] + atomicAdd(cursor + e, 1) : -1;
     pos[pair] = where;
   }
   __syncthreads();
+  if (where < 0) return;                         // an identity expert has no row
   const T* src = h + (pair / top) * ldh;
   T* dst = xs + (long)where * n;
   constexpr int PER = 16 / sizeof(T);
@@ -1162,19 +1192,21 @@ int lbk_masked_attention(const void* q, long ldq, const void* kbase, const void*
   LAUNCH_END();
 }
 
-int lbk_moe_topk(const float* z, long ldz, const float* bias, int mode, int E, int top, float rscale, int* idx, float* wts, int* counts,
-                 long tokens, cudaStream_t s) {
+int lbk_moe_topk(const float* z, long ldz, const float* bias, const float* corr, int mode, int E, int real, int top, float rscale, int* idx,
+                 float* wts, int* counts, float* keep, long tokens, cudaStream_t s) {
   if (tokens == 0) return 0;
-  if (top > E || (size_t)E * sizeof(float) > 12 * 1024) return -1;
   const int warps = 4;
-  moe_topk_kernel<<<(unsigned)((tokens + warps - 1) / warps), warps * 32, (size_t)warps * E * sizeof(float), s>>>(z, ldz, bias, mode, E, top, rscale,
-                                                                                                               idx, wts, counts, tokens);
+  const size_t smem = (size_t)warps * E * sizeof(float) * (mode == 3 ? 2 : 1);
+  if (top > E || real < 1 || real > E || smem > 48 * 1024) return -1;
+  moe_topk_kernel<<<(unsigned)((tokens + warps - 1) / warps), warps * 32, smem, s>>>(z, ldz, bias, corr, mode, E, real, top, rscale, idx, wts, counts,
+                                                                                    keep, tokens);
   LAUNCH_END();
 }
 
 int lbk_moe_pairs(const void* h, long ldh, const void* wgu, const void* wd, const int* idx, const float* wts, void* a, float* out,
-                  long tokens, int ff, int n, int top, int act, float limit, int win, int dtype, cudaStream_t s) {
+                  long tokens, int E, int ff, int n, int top, int act, int gated, float limit, int win, int dtype, cudaStream_t s) {
   if (tokens == 0) return 0;
+  if (act == 5 && !gated) return -1;
   const size_t smem1 = (size_t)n * sizeof(float), smem2 = (size_t)top * ff * sizeof(float);
   if (smem1 > 200 * 1024 || smem2 > 200 * 1024) return -1;
   const long pairs = tokens * top;
@@ -1184,13 +1216,13 @@ int lbk_moe_pairs(const void* h, long ldh, const void* wgu, const void* wd, cons
   if (dtype) {
     if (smem1 > 48 * 1024) cudaFuncSetAttribute(moe_pair_gateup_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
     if (smem2 > 48 * 1024) cudaFuncSetAttribute(moe_pair_down_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);
-    moe_pair_gateup_kernel<bf16><<<dim3((unsigned)pairs, sy1), 256, smem1, s>>>((const bf16*)h, ldh, (const bf16*)wgu, idx, wts, win, (bf16*)a, ff, n, top, act, limit);
-    moe_pair_down_kernel<bf16><<<dim3((unsigned)tokens, sy2), 256, smem2, s>>>((const bf16*)a, (const bf16*)wd, idx, wts, win, out, ff, n, top);
+    moe_pair_gateup_kernel<bf16><<<dim3((unsigned)pairs, sy1), 256, smem1, s>>>((const bf16*)h, ldh, (const bf16*)wgu, idx, wts, win, (bf16*)a, E, ff, n, top, act, gated, limit);
+    moe_pair_down_kernel<bf16><<<dim3((unsigned)tokens, sy2), 256, smem2, s>>>((const bf16*)a, (const bf16*)wd, idx, wts, win, out, E, ff, n, top);
   } else {
     if (smem1 > 48 * 1024) cudaFuncSetAttribute(moe_pair_gateup_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
     if (smem2 > 48 * 1024) cudaFuncSetAttribute(moe_pair_down_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);
-    moe_pair_gateup_kernel<float><<<dim3((unsigned)pairs, sy1), 256, smem1, s>>>((const float*)h, ldh, (const float*)wgu, idx, wts, win, (float*)a, ff, n, top, act, limit);
-    moe_pair_down_kernel<float><<<dim3((unsigned)tokens, sy2), 256, smem2, s>>>((const float*)a, (const float*)wd, idx, wts, win, out, ff, n, top);
+    moe_pair_gateup_kernel<float><<<dim3((unsigned)pairs, sy1), 256, smem1, s>>>((const float*)h, ldh, (const float*)wgu, idx, wts, win, (float*)a, E, ff, n, top, act, gated, limit);
+    moe_pair_down_kernel<float><<<dim3((unsigned)tokens, sy2), 256, smem2, s>>>((const float*)a, (const float*)wd, idx, wts, win, out, E, ff, n, top);
   }
   LAUNCH_END();
 }
@@ -1201,8 +1233,8 @@ int lbk_moe_sort(const void* h, long ldh, const int* idx, const int* counts, int
   if (E > 1024 || align < 1) return -1;
   moe_offsets_kernel<<<1, 256, 0, s>>>(counts, offsets, cursor, E, align, tile_group, tiles);
   const unsigned pairs = (unsigned)(tokens * top);
-  if (dtype) moe_scatter_kernel<bf16><<<pairs, 128, 0, s>>>((const bf16*)h, ldh, idx, offsets, cursor, pos, (bf16*)xs, n, top, wts);
-  else moe_scatter_kernel<float><<<pairs, 128, 0, s>>>((const float*)h, ldh, idx, offsets, cursor, pos, (float*)xs, n, top, wts);
+  if (dtype) moe_scatter_kernel<bf16><<<pairs, 128, 0, s>>>((const bf16*)h, ldh, idx, offsets, cursor, pos, (bf16*)xs, E, n, top, wts);
+  else moe_scatter_kernel<float><<<pairs, 128, 0, s>>>((const float*)h, ldh, idx, offsets, cursor, pos, (float*)xs, E, n, top, wts);
   LAUNCH_END();
 }
 

@@ -1,7 +1,7 @@
 // Kernels of decoders whose attention layers see the whole past of a sequence through a paged key/value cache:
 //   * post-norm residual: x <- rmsnorm(alpha * x + sublayer output) * (1 + w) on the fp32 residual, with the compute-dtype copy
 //     that the next sublayer's products read (the sublayer output may be a dense matrix plus rows gathered from a matrix of
-//     expert outputs sorted by expert);
+//     expert outputs sorted by expert), and its outer form x <- x + rmsnorm(sublayer output) * (1 + w);
 //   * query / key / value preparation in one pass: per-channel causal convolution over time (tails carried per sequence),
 //     per-head RMS norm of queries and keys with a weight shared by the heads, rotary positions on the leading channels,
 //     unit-RMS values, keys and values written into their page;
@@ -52,9 +52,10 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 }
 
 // ------------------------------------------------------------------------------------------------------------------
-// Post-norm residual.  v = alpha * x + y1 + y2', r = 1 / sqrt(mean(v^2) + eps), out = v * r * (1 + w); `xout` (fp32, may
-// be x itself) and `h` (T) receive it when given.  y1 [rows, n] (Ty) and y2 (fp32) are optional; with `pos` [rows, top]
-// y2' = sum_k cw[r, k] * y2[pos[r, k]] (cw absent: 1), else y2' = y2[r].  One block per row; the row is staged in shared memory.
+// Post-norm residual.  v = (alpha + keep[row]) * x + sigmoid(gate[row]) * y1 + y2', o = v / sqrt(mean(v^2) + eps) * (1 + w) *
+// out_scale, out = o or — `outer` — x + o; `xout` (fp32, may be x itself) and `h` (T) receive it when given.  y1 [rows, n] (Ty) and
+// y2 (fp32) are optional (gate absent: y1 as it is; keep absent: 0); with `pos` [rows, top] y2' = sum_k cw[r, k] * y2[pos[r, k]]
+// (cw absent: 1; an entry -1 contributes nothing), else y2' = y2[r].  One block per row; the row is staged in shared memory.
 // ------------------------------------------------------------------------------------------------------------------
 __device__ __forceinline__ float4 ld4f(const float* p) { return *reinterpret_cast<const float4*>(p); }
 __device__ __forceinline__ float4 ld4f(const bf16* p) {
@@ -75,9 +76,12 @@ __device__ __forceinline__ void st4f(bf16* p, float4 v) {
 template <typename T, typename Ty, int ITEMS>
 __global__ void postnorm_residual_vec_kernel(const float* xin, float* xout, const Ty* __restrict__ y1, long ldy1, const float* __restrict__ y2,
                                              long ldy2, const int* __restrict__ pos, const float* __restrict__ cw, int top, float alpha,
-                                             const T* __restrict__ w, float eps, T* __restrict__ h, long ldh, int n) {
+                                             const float* __restrict__ gate, long ldgate, const float* __restrict__ keep, int outer,
+                                             float out_scale, const T* __restrict__ w, float eps, T* __restrict__ h, long ldh, int n) {
   __shared__ float red[32];
   const long row = blockIdx.x;
+  const float g1 = gate ? 1.f / (1.f + expf(-gate[row * ldgate])) : 1.f;
+  if (keep) alpha += keep[row];
   const int quads = n / 4;
   float4 v[ITEMS];
   float ss = 0.f;
@@ -88,12 +92,14 @@ __global__ void postnorm_residual_vec_kernel(const float* xin, float* xout, cons
     if (i < quads * 4) {
       float4 a = ld4f(xin + row * n + i);
       a.x *= alpha; a.y *= alpha; a.z *= alpha; a.w *= alpha;
-      if (y1) { const float4 b = ld4f(y1 + row * ldy1 + i); a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w; }
+      if (y1) { const float4 b = ld4f(y1 + row * ldy1 + i); a.x += g1 * b.x; a.y += g1 * b.y; a.z += g1 * b.z; a.w += g1 * b.w; }
       if (y2) {
         if (pos) {
           for (int k = 0; k < top; ++k) {
+            const int pk = pos[row * top + k];
+            if (pk < 0) continue;
             const float c = cw ? cw[row * top + k] : 1.f;
-            const float4 b = ld4f(y2 + (long)pos[row * top + k] * ldy2 + i);
+            const float4 b = ld4f(y2 + (long)pk * ldy2 + i);
             a.x += c * b.x; a.y += c * b.y; a.z += c * b.z; a.w += c * b.w;
           }
         } else {
@@ -106,13 +112,14 @@ __global__ void postnorm_residual_vec_kernel(const float* xin, float* xout, cons
     }
   }
   ss = block_sum(ss, red);
-  const float r = 1.f / sqrtf(ss / (float)n + eps);
+  const float r = 1.f / sqrtf(ss / (float)n + eps) * out_scale;
 #pragma unroll
   for (int it = 0; it < ITEMS; ++it) {
     const int i = (threadIdx.x + it * blockDim.x) * 4;
     if (i < quads * 4) {
       const float4 ww = ld4f(w + i);
-      const float4 o = make_float4(v[it].x * r * (1.f + ww.x), v[it].y * r * (1.f + ww.y), v[it].z * r * (1.f + ww.z), v[it].w * r * (1.f + ww.w));
+      float4 o = make_float4(v[it].x * r * (1.f + ww.x), v[it].y * r * (1.f + ww.y), v[it].z * r * (1.f + ww.z), v[it].w * r * (1.f + ww.w));
+      if (outer) { const float4 xr = ld4f(xin + row * n + i); o.x += xr.x; o.y += xr.y; o.z += xr.z; o.w += xr.w; }
       if (xout) st4f(xout + row * n + i, o);
       if (h) st4f(h + row * ldh + i, o);
     }
@@ -122,17 +129,23 @@ __global__ void postnorm_residual_vec_kernel(const float* xin, float* xout, cons
 template <typename T, typename Ty>
 __global__ void postnorm_residual_kernel(const float* xin, float* xout, const Ty* __restrict__ y1, long ldy1, const float* __restrict__ y2,
                                          long ldy2, const int* __restrict__ pos, const float* __restrict__ cw, int top, float alpha,
-                                         const T* __restrict__ w, float eps, T* __restrict__ h, long ldh, int n) {
+                                         const float* __restrict__ gate, long ldgate, const float* __restrict__ keep, int outer,
+                                         float out_scale, const T* __restrict__ w, float eps, T* __restrict__ h, long ldh, int n) {
   extern __shared__ float sm[];
   __shared__ float red[32];
   const long row = blockIdx.x;
+  const float g1 = gate ? 1.f / (1.f + expf(-gate[row * ldgate])) : 1.f;
+  if (keep) alpha += keep[row];
   float ss = 0.f;
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
     float v = alpha * xin[row * n + i];
-    if (y1) v += ldf(y1 + row * ldy1 + i);
+    if (y1) v += g1 * ldf(y1 + row * ldy1 + i);
     if (y2) {
       if (pos) {
-        for (int k = 0; k < top; ++k) v += (cw ? cw[row * top + k] : 1.f) * y2[(long)pos[row * top + k] * ldy2 + i];
+        for (int k = 0; k < top; ++k) {
+          const int pk = pos[row * top + k];
+          if (pk >= 0) v += (cw ? cw[row * top + k] : 1.f) * y2[(long)pk * ldy2 + i];
+        }
       } else {
         v += y2[row * ldy2 + i];
       }
@@ -141,9 +154,10 @@ __global__ void postnorm_residual_kernel(const float* xin, float* xout, const Ty
     ss += v * v;
   }
   ss = block_sum(ss, red);
-  const float r = 1.f / sqrtf(ss / (float)n + eps);
+  const float r = 1.f / sqrtf(ss / (float)n + eps) * out_scale;
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const float o = sm[i] * r * (1.f + ldf(w + i));
+    float o = sm[i] * r * (1.f + ldf(w + i));
+    if (outer) o += xin[row * n + i];
     if (xout) xout[row * n + i] = o;
     if (h) stf(h + row * ldh + i, o);
   }
@@ -776,8 +790,9 @@ __global__ void talk_attention_merge_kernel(const float* __restrict__ part, cons
 extern "C" {
 
 int lbp_postnorm_residual(const float* xin, float* xout, const void* y1, long ldy1, int y1dtype, const float* y2, long ldy2,
-                          const int* pos, const float* cw, int top, float alpha, const void* w, float eps, void* h, long ldh,
-                          long rows, int n, int dtype, cudaStream_t s) {
+                          const int* pos, const float* cw, int top, float alpha, const float* gate, long ldgate, const float* keep,
+                          int outer, float out_scale, const void* w, float eps, void* h, long ldh, long rows, int n, int dtype,
+                          cudaStream_t s) {
   if (rows == 0) return 0;
   const size_t smem = (size_t)n * sizeof(float);
   if (smem > 160 * 1024) return -1;
@@ -790,7 +805,7 @@ int lbp_postnorm_residual(const float* xin, float* xout, const void* y1, long ld
     int vthreads = (((quads + items - 1) / items + 31) / 32) * 32;
     if (vthreads > 1024) vthreads = 1024;
 #define PNV(TT, TY, IT) postnorm_residual_vec_kernel<TT, TY, IT><<<(unsigned)rows, vthreads, 0, s>>>(xin, xout, (const TY*)y1, ldy1, y2, ldy2, pos, cw, top, \
-        alpha, (const TT*)w, eps, (TT*)h, ldh, n)
+        alpha, gate, ldgate, keep, outer, out_scale, (const TT*)w, eps, (TT*)h, ldh, n)
 #define PNV2(TT, TY) { if (items == 1) PNV(TT, TY, 1); else PNV(TT, TY, 2); }
     if (dtype) { if (y1dtype) PNV2(bf16, bf16) else PNV2(bf16, float) }
     else { if (y1dtype) return -1; PNV2(float, float) }
@@ -802,7 +817,7 @@ int lbp_postnorm_residual(const float* xin, float* xout, const void* y1, long ld
 #define PN(TT, TY) { \
     if (smem > 48 * 1024) cudaFuncSetAttribute(postnorm_residual_kernel<TT, TY>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     postnorm_residual_kernel<TT, TY><<<(unsigned)rows, threads, smem, s>>>(xin, xout, (const TY*)y1, ldy1, y2, ldy2, pos, cw, top, alpha, \
-                                                                           (const TT*)w, eps, (TT*)h, ldh, n); }
+                                                                           gate, ldgate, keep, outer, out_scale, (const TT*)w, eps, (TT*)h, ldh, n); }
   if (dtype) { if (y1dtype) PN(bf16, bf16) else PN(bf16, float) }
   else { if (y1dtype) return -1; PN(float, float) }
 #undef PN

@@ -62,6 +62,21 @@ class KvExt:
         self.ext_seq = packed[3 * B + 1:]
 
 
+class PageExt:
+    """Row layout of a step that reads every cached position of its sequences: per sequence the rows of the positions
+    ``0 … past + new − 1``."""
+
+    def __init__(self, rb: "RaggedBatch"):
+        lens = [p + n for p, n in zip(rb.past_list, rb.lens)]
+        self.offsets = [0]
+        for n in lens:
+            self.offsets.append(self.offsets[-1] + n)
+        self.rows = self.offsets[-1]
+        packed = torch.tensor(self.offsets, dtype=torch.int32).to(rb.device, non_blocking=True)
+        self.ext_off = packed
+        self.ext_seq = torch.repeat_interleave(torch.arange(rb.B, dtype=torch.int32), torch.tensor(lens)).to(rb.device, non_blocking=True)
+
+
 class RaggedBatch:
     def __init__(self, lens: Sequence[int], slots: Sequence[int], past: Sequence[int], device):
         assert len(lens) == len(slots) == len(past) and all(n > 0 for n in lens)
@@ -80,6 +95,7 @@ class RaggedBatch:
         self.tok_seq = packed[3 * B + 1:]
         self._ext: Dict[int, WindowExt] = {}
         self._kv_ext: Dict[tuple, KvExt] = {}
+        self._page_ext = None
         self._tiles: Dict[int, tuple] = {}
 
     def ext(self, window: int) -> WindowExt:
@@ -93,6 +109,11 @@ class RaggedBatch:
         if key not in self._kv_ext:
             self._kv_ext[key] = KvExt(self, key)
         return self._kv_ext[key]
+
+    def page_ext(self) -> PageExt:
+        if self._page_ext is None:
+            self._page_ext = PageExt(self)
+        return self._page_ext
 
     def query_tiles(self, size: int):
         """Tiles of ``size`` consecutive new tokens of one sequence: (sequence of every tile, its first token) on the device."""

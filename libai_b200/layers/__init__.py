@@ -17,9 +17,9 @@ __all__ = [
 ]
 from .delta_rule import GatedDeltaMixer
 from .hyper_connections import HyperConnection
-from .latent_attention import LatentAttention
+from .latent_attention import LatentAttention, PagedLatentAttention
 from .layer_norm import DynamicTanh
 from .linear_attention import DecayLinearAttention
-from .moe import GatedFeedForward, MoEFeedForward
+from .moe import FeedForward, GatedFeedForward, MoEFeedForward
 from .paged_attention import PagedAttention
 from .ring_attention import RingAttention

@@ -7,6 +7,7 @@ from .llama_model import LlamaForCausalLM, LlamaModel
 from .resmlp import ResMLP
 from .salizen_model import SalizenForCausalLM, SalizenModel
 from .roberta_model import RobertaForCausalLM, RobertaForPreTraining, RobertaModel
+from .voduzen_model import VoduzenForCausalLM, VoduzenModel
 from .zubarax_model import ZubaraxForCausalLM, ZubaraxModel
 from .swin_transformer import SwinTransformer
 from .swin_transformer_v2 import SwinTransformerV2
@@ -22,5 +23,5 @@ __all__ = [
     "VisionTransformer", "SwinTransformer", "SwinTransformerV2", "ResMLP",
     "LlamaModel", "LlamaForCausalLM",
     "BumodraModel", "BumodraForCausalLM", "NefelornModel", "NefelornForCausalLM",
-    "SalizenModel", "SalizenForCausalLM", "ZubaraxModel", "ZubaraxForCausalLM",
+    "SalizenModel", "SalizenForCausalLM", "VoduzenModel", "VoduzenForCausalLM", "ZubaraxModel", "ZubaraxForCausalLM",
 ]

@@ -28,8 +28,8 @@ from torch import nn
 from libai_b200.config import configurable
 from libai_b200.inference.ragged import RaggedBatch
 from libai_b200.inference.state_cache import SequenceStateCache
-from libai_b200.layers import DynamicTanh, MoEFeedForward, RingAttention
-from libai_b200.layers._param import create_parameter, normal_init, xavier_normal_
+from libai_b200.layers import DynamicTanh, FeedForward, MoEFeedForward, RingAttention
+from libai_b200.layers._param import create_parameter, normal_init
 from libai_b200.ops import kv_functional as KF
 from libai_b200.ops import seq_functional as SF
 
@@ -51,21 +51,6 @@ def build_ring_mixer(kind: str, width: int, m: dict, eps: float, layer_idx: int)
     raise ValueError(f"unknown mixer type {kind!r}")
 
 
-class GeluFF(nn.Module):
-    """``W_down act(W_up h)`` without biases."""
-
-    def __init__(self, width, ff, act="gelu", *, layer_idx=0):
-        super().__init__()
-        self.act = act
-        self.up = create_parameter((ff, width), xavier_normal_, layer_idx=layer_idx)
-        self.down = create_parameter((width, ff), xavier_normal_, layer_idx=layer_idx)
-
-    def forward(self, h):
-        u = KF.linear(h, self.up)
-        KF.act_rows(u, u, KF.ACTS[self.act])
-        return KF.linear_f32(u, self.down)
-
-
 class SandwichBlock(nn.Module):
     """``x ← x + n1b(mixer(n1(x)))``, ``x ← x + n2b(ff(n2(x)))`` on the fp32 stream ``x``; the opening norm of a sublayer is
     applied by the kernel that closes the sublayer before it, so a block receives ``h = n1(x)`` and returns the next block's."""
@@ -81,7 +66,7 @@ class SandwichBlock(nn.Module):
             self.norm2, self.norm2b = mk(), mk()
             kind_ff = mlp_cfg.get("kind", "dense")
             if kind_ff == "dense":
-                self.mlp = GeluFF(width, mlp_cfg["ff"], layer_idx=layer_idx)
+                self.mlp = FeedForward(width, mlp_cfg["ff"], layer_idx=layer_idx)
             elif kind_ff == "moe":
                 r = mlp_cfg["router"]
                 self.mlp = MoEFeedForward(width, mlp_cfg["expert"]["ff"], r["experts"], r["top"], router_scale=r.get("scale", 1.0),

@@ -49,10 +49,18 @@ def _zubarax():
     return ZubaraxForCausalLM, ZubaraxLoader, {}
 
 
+def _voduzen():
+    from libai_b200.models import VoduzenForCausalLM
+    from .voduzen_loader import VoduzenLoader
+
+    return VoduzenForCausalLM, VoduzenLoader, {}
+
+
 ARCHITECTURES = {
     "bumodra": _bumodra,
     "nefelorn": _nefelorn,
     "salizen": _salizen,
+    "voduzen": _voduzen,
     "zubarax": _zubarax,
     "llama": _llama, "llamaforcausallm": _llama,
 }
@@ -60,7 +68,7 @@ ARCHITECTURES = {
 
 # native libraries (``libai_b200.ops.build``) that a model's generation path launches besides the GEMM library ``_C``
 NATIVE_LIBS = {"bumodra": ["_C_seq"], "nefelorn": ["_C_kv"], "salizen": ["_C_kv", "_C_lin"],
-               "zubarax": ["_C_kv", "_C_lin"]}
+               "voduzen": ["_C_kv"], "zubarax": ["_C_kv", "_C_lin"]}
 
 
 def native_libs_of(path: str, dtype=torch.bfloat16):

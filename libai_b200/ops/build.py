@@ -31,8 +31,8 @@ SEQ_SO_PATH = os.path.join(ROOT, "_C_seq.so")
 SEQ_CU_SOURCES = ["seq_mixers.cu"]
 SEQ_CPP_SOURCES = ["seq_bindings.cpp"]
 KV_SO_PATH = os.path.join(ROOT, "_C_kv.so")
-KV_CU_SOURCES = ["kv_mixers.cu", "paged_mixers.cu"]
-KV_CPP_SOURCES = ["kv_bindings.cpp"]
+KV_CU_SOURCES = ["kv_mixers.cu", "paged_mixers.cu", "latent_mixers.cu"]
+KV_CPP_SOURCES = ["kv_bindings.cpp", "latent_bindings.cpp"]
 LIN_SO_PATH = os.path.join(ROOT, "_C_lin.so")
 LIN_CU_SOURCES = ["lin_mixers.cu"]
 LIN_CPP_SOURCES = ["lin_bindings.cpp"]

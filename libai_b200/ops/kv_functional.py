@@ -336,27 +336,40 @@ def ring_attention(q, ring, first, gate, rb, y, H: int, G: int, D: int, V: int, 
 
 
 # ------------------------------------------------------------------------------------------------------ mixture of experts
-ROUTE_SIGMOID, ROUTE_SOFTMAX, ROUTE_SIGMOID_RAW = 0, 1, 2
+ROUTE_SIGMOID, ROUTE_SOFTMAX, ROUTE_SIGMOID_RAW, ROUTE_SOFTMAX_ALL = 0, 1, 2, 3
 
 
-def moe_route(h, wr, top: int, rscale: float, counts=None, bias=None, mode: int = ROUTE_SIGMOID):
+def moe_route(h, wr, top: int, rscale: float, counts=None, bias=None, mode: int = ROUTE_SIGMOID, *, z=None, choices: Optional[int] = None,
+              experts: Optional[int] = None, correction=None, keep=None):
     """Router on the fp32 logits ``z = W_r h`` (``+ bias``, fp32 ``[E]``).  ``ROUTE_SIGMOID``: the ``top`` largest
     ``s = sigmoid(z)``, weights ``s / (Σ s + 1e-20) · rscale``; ``ROUTE_SOFTMAX``: the ``top`` largest logits, weights = softmax
     over the chosen logits only, times ``rscale``; ``ROUTE_SIGMOID_RAW``: the ``top`` largest ``s = sigmoid(z)``, weights
-    ``s · rscale`` (not normalised).  Ties go to the lower index.  Returns ``idx`` int32 and ``wts`` fp32, both
-    ``[tokens, top]``; ``counts`` (int32 ``[E]``, zeroed by the caller) receives the number of tokens of every expert."""
+    ``s · rscale`` (not normalised); ``ROUTE_SOFTMAX_ALL``: ``s = softmax(z)`` over all choices, the ``top`` largest
+    ``s + correction`` (fp32 ``[E]``), weights ``s · rscale``.  Ties go to the lower index.  Returns ``idx`` int32 and ``wts`` fp32, both
+    ``[tokens, top]``; ``counts`` (int32 ``[E]``, zeroed by the caller) receives the number of tokens of every expert.
+
+    ``z``: the logits when the caller has them already (``choices``: how many of their leading columns count).  Choices at or
+    above ``experts`` are identity experts, whose output is the token itself: they are not counted, and the sum of their weights
+    goes to ``keep`` (fp32 ``[tokens]``)."""
     T = h.shape[0]
     idx = torch.empty(T, top, dtype=torch.int32, device=h.device)
     wts = torch.empty(T, top, dtype=torch.float32, device=h.device)
-    if _native(h):
+    if z is None:
         z = router_logits(h, wr)
+    E = z.shape[1] if choices is None else int(choices)
+    real = E if experts is None else int(experts)
+    if _native(h):
         count_launch()
-        load_kv_ext().moe_topk(z, bias, mode, top, float(rscale), idx, wts, counts)
+        load_kv_ext().moe_topk(z, bias, mode, top, float(rscale), idx, wts, counts, correction, E, real, keep)
         return idx, wts
-    z = F.linear(h.float(), wr.float())
+    z = z[:, :E]
     if bias is not None:
         z = z + bias.float()
-    if mode == ROUTE_SOFTMAX:
+    if mode == ROUTE_SOFTMAX_ALL:
+        s = torch.softmax(z, -1)
+        ti = (s + correction.float() if correction is not None else s).topk(top, -1).indices
+        w = s.gather(1, ti) * rscale
+    elif mode == ROUTE_SOFTMAX:
         tv, ti = z.topk(top, -1)
         w = torch.softmax(tv, -1) * rscale
     else:
@@ -365,7 +378,9 @@ def moe_route(h, wr, top: int, rscale: float, counts=None, bias=None, mode: int 
     idx.copy_(ti)
     wts.copy_(w)
     if counts is not None:
-        counts.add_(torch.bincount(ti.reshape(-1), minlength=counts.numel()).to(counts.dtype))
+        counts.add_(torch.bincount(ti.reshape(-1), minlength=E)[: counts.numel()].to(counts.dtype))
+    if keep is not None:
+        keep.copy_((w * (ti >= real)).sum(1))
     return idx, wts
 
 
@@ -383,46 +398,50 @@ def router_logits(h, wr):
     return F.linear(h.float(), wr.float())
 
 
-def moe_pairs(h, wgu, wd, idx, wts, act: int, limit: float = 0.0, weight_input: bool = False):
+def moe_pairs(h, wgu, wd, idx, wts, act: int, limit: float = 0.0, weight_input: bool = False, gated: bool = True):
     """Experts for few tokens: every (token, chosen expert) pair reads its expert's matrices.  ``wgu`` ``[E, 2·ff, width]``
-    (gate rows, then up rows), ``wd`` ``[E, width, ff]``.  Returns ``Σ_k wts[t,k] · W_down,k (act(W_gate,k h) · W_up,k h)`` as
+    (gate rows, then up rows; ``gated=False``: ``[E, ff, width]`` and ``act(W_up h)``), ``wd`` ``[E, width, ff]``; pairs whose expert
+    number is ``E`` or more contribute nothing.  Returns ``Σ_k wts[t,k] · W_down,k (act(W_gate,k h) · W_up,k h)`` as
     fp32 ``[tokens, width]``; with ``weight_input`` the weight multiplies the expert's input instead (``wts[t,k] · h`` rounded to
     the compute dtype) and the outputs are summed."""
     T, n = h.shape
-    top, ff = idx.shape[1], wgu.shape[1] // 2
+    top, ff = idx.shape[1], wd.shape[2]
     out = torch.empty(T, n, dtype=torch.float32, device=h.device)
     if _native(h):
         count_launch(2)
         a = torch.empty(T * top, ff, dtype=h.dtype, device=h.device)
-        load_kv_ext().moe_pairs(h, wgu, wd, idx, wts, a, out, act, float(limit), bool(weight_input))
+        load_kv_ext().moe_pairs(h, wgu, wd, idx, wts, a, out, act, float(limit), bool(weight_input), bool(gated))
         return out
     for t in range(T):
         acc = torch.zeros(n)
         for k in range(top):
             e = int(idx[t, k])
+            if e >= wd.shape[0]:
+                continue
             hin = (wts[t, k] * h[t].float()).to(h.dtype).float() if weight_input else h[t].float()
             gu = wgu[e].float() @ hin
-            a = _gated_pair(gu[:ff], gu[ff:], act, limit).to(h.dtype).float()
+            a = (_gated_pair(gu[:ff], gu[ff:], act, limit) if gated else _act(gu, act)).to(h.dtype).float()
             acc += (1.0 if weight_input else wts[t, k]) * (wd[e].float() @ a)
         out[t] = acc
     return out
 
 
-def moe_sorted(h, wgu, wd, idx, counts, act: int, limit: float = 0.0, in_wts=None):
+def moe_sorted(h, wgu, wd, idx, counts, act: int, limit: float = 0.0, in_wts=None, gated: bool = True):
     """Experts for many tokens: the rows are copied into a matrix sorted by expert, every expert runs as two dense products on
     its row range, and the caller gathers the weighted sum (:func:`dyt_residual` with ``pos``).  Returns
     ``(ys fp32 [rows, width], pos int32 [tokens, top])``: the output row of pair (t, k) is ``ys[pos[t, k]]``.  With ``in_wts``
     (fp32 ``[tokens, top]``) the copied row of pair (t, k) is ``in_wts[t, k] · h[t]``: routing weights on the experts' inputs.
+    ``gated`` as in :func:`moe_pairs`; a pair whose expert number is ``E`` or more has no row, ``pos[t, k] = −1``.
 
     bf16 on the GPU: every expert's range starts on a multiple of 128 rows and each product is ONE launch of the tcgen05 GEMM
     in its grouped mode (the expert of every 128-row block is a device-side list), so nothing is read back by the host and the
     step can be captured.  Otherwise (fp32, CPU) the per-expert row counts are read back and the experts run one by one."""
     T, n = h.shape
-    top, E, ff = idx.shape[1], wgu.shape[0], wgu.shape[1] // 2
+    top, E, ff, ups = idx.shape[1], wgu.shape[0], wd.shape[2], wgu.shape[1]
     P = T * top
     dev = h.device
     pos = torch.empty(T, top, dtype=torch.int32, device=dev)
-    if _native(h) and h.dtype == torch.bfloat16 and n % 8 == 0 and ff % 8 == 0 and E * max(2 * ff, n) < 2 ** 31:
+    if _native(h) and h.dtype == torch.bfloat16 and n % 8 == 0 and ff % 8 == 0 and E * max(ups, n) < 2 ** 31:
         from . import load_ext
 
         rows = (P + E * 127 + 127) // 128 * 128
@@ -431,10 +450,10 @@ def moe_sorted(h, wgu, wd, idx, counts, act: int, limit: float = 0.0, in_wts=Non
         groups = meta[2 * E + 1:]
         count_launch(5)
         load_kv_ext().moe_sort(h, idx, counts, meta[: E + 1], meta[E + 1: 2 * E + 1], pos, xs, 128, groups, in_wts)
-        gu = torch.empty(rows, 2 * ff, dtype=h.dtype, device=dev)
+        gu = torch.empty(rows, ups, dtype=h.dtype, device=dev)
         load_ext().gemm_grouped_blocks(xs, wgu.detach(), groups, gu)
-        a = torch.empty(rows, ff, dtype=h.dtype, device=dev)
-        act_rows(gu, a, act, gated=True, limit=limit)
+        a = torch.empty(rows, ff, dtype=h.dtype, device=dev) if gated else gu
+        act_rows(gu, a, act, gated=gated, limit=limit)
         ys = torch.empty(rows, n, dtype=torch.float32, device=dev)
         load_ext().gemm_grouped_blocks(a, wd.detach(), groups, ys)
         return ys, pos
@@ -448,12 +467,16 @@ def moe_sorted(h, wgu, wd, idx, counts, act: int, limit: float = 0.0, in_wts=Non
         order = torch.sort(idx.reshape(-1).long(), stable=True).indices
         pos.view(-1)[order] = torch.arange(P, dtype=torch.int32)
         xs.copy_(h[order // top] if in_wts is None else in_wts.reshape(-1)[order][:, None] * h[order // top].float())
-        cnt = torch.bincount(idx.reshape(-1).long(), minlength=E).tolist()
-    gu = torch.empty(P, 2 * ff, dtype=h.dtype, device=dev)
-    a = torch.empty(P, ff, dtype=h.dtype, device=dev)
-    ys = torch.empty(P, n, dtype=torch.float32, device=dev)
+        pos.masked_fill_(idx >= E, -1)
+        cnt = torch.bincount(idx.reshape(-1).long(), minlength=E)[:E].tolist()
+    if sum(cnt) < P:                                            # pairs of identity experts have no rows
+        P = sum(cnt)
+        xs = xs[:max(P, 1)]
+    gu = torch.empty(xs.shape[0], ups, dtype=h.dtype, device=dev)
+    a = torch.empty(xs.shape[0], ff, dtype=h.dtype, device=dev) if gated else gu
+    ys = torch.empty(xs.shape[0], n, dtype=torch.float32, device=dev)
     _grouped_products(xs, wgu, cnt, gu, False)
-    act_rows(gu, a, act, gated=True, limit=limit)
+    act_rows(gu, a, act, gated=gated, limit=limit)
     _grouped_products(a, wd, cnt, ys, False)
     return ys, pos
 

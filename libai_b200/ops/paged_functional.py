@@ -20,31 +20,45 @@ def _native(t: torch.Tensor) -> bool:
 
 
 # ------------------------------------------------------------------------------------------------------------ residual
-def postnorm_residual(x, w, eps: float, *, alpha: float = 1.0, y=None, y2=None, pos=None, cw=None, h=None, inplace: bool = True):
+def postnorm_residual(x, w, eps: float, *, alpha: float = 1.0, y=None, y2=None, pos=None, cw=None, h=None, inplace: bool = True,
+                      gate=None, keep=None, outer: bool = False, out_scale: float = 1.0):
     """``v = alpha · x + y + y2'``, ``out = v / sqrt(mean(v²) + eps) · (1 + w)`` on the fp32 residual ``x`` ``[rows, width]``.
     ``y`` ``[rows, width]`` (fp32 or the compute dtype) and ``y2`` (fp32) are optional sublayer outputs; with ``pos``
     ``[rows, top]`` the second one is gathered, ``y2' = Σ_k cw[r, k] · y2[pos[r, k]]`` (``cw`` absent: plain sum), which is how
-    expert outputs sorted by expert come back to their tokens.  ``out`` replaces ``x`` (``inplace``) and is also written to
-    ``h`` (compute dtype) when given — the copy the next sublayer's products read."""
+    expert outputs sorted by expert come back to their tokens (an entry −1 of ``pos`` contributes nothing).  ``out`` replaces
+    ``x`` (``inplace``) and is also written to ``h`` (compute dtype) when given — the copy the next sublayer's products read.
+    Further terms: ``gate`` (fp32 ``[rows]``, may be a column of a matrix) multiplies ``y`` by its sigmoid; ``keep`` (fp32 ``[rows]``)
+    adds ``keep[r] · x`` to ``v``; ``out_scale`` multiplies the normed row; ``outer`` adds ``x`` after the norm (a norm on the
+    sublayer's output only, see :func:`outnorm_residual`)."""
     if _native(x):
         count_launch()
-        load_kv_ext().postnorm_residual(x, x if inplace else None, y, y2, pos, cw, float(alpha), w, float(eps), h)
+        load_kv_ext().postnorm_residual(x, x if inplace else None, y, y2, pos, cw, float(alpha), w, float(eps), h, gate, keep, outer, float(out_scale))
         return x
     v = alpha * x
+    if keep is not None:
+        v = v + keep[:, None] * x
     if y is not None:
-        v = v + y.float()
+        v = v + (torch.sigmoid(gate)[:, None] * y.float() if gate is not None else y.float())
     if y2 is not None:
         if pos is not None:
-            g = y2[pos.long()]
-            v = v + (g * cw[:, :, None] if cw is not None else g).sum(1)
+            g = y2[pos.clamp(min=0).long()] * (cw[:, :, None] if cw is not None else 1.0)
+            v = v + g.masked_fill((pos < 0)[:, :, None], 0.0).sum(1)
         else:
             v = v + y2
-    out = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * (1.0 + w.float())
+    out = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * (1.0 + w.float()) * out_scale
+    if outer:
+        out = x + out
     if inplace:
         x.copy_(out)
     if h is not None:
         h.copy_(out)
     return x
+
+
+def outnorm_residual(x, w, eps: float, *, y=None, y2=None, pos=None, cw=None, gate=None, keep=None, h=None):
+    """``x ← x + v / sqrt(mean(v²) + eps) · (1 + w)`` with ``v = sigmoid(gate) · y + y2' + keep · x`` (the terms of
+    :func:`postnorm_residual`): the norm is on the sublayer's output, the residual itself is never normed."""
+    return postnorm_residual(x, w, eps, alpha=0.0, y=y, y2=y2, pos=pos, cw=cw, h=h, gate=gate, keep=keep, outer=True)
 
 
 # ------------------------------------------------------------------------------------------------- query / key / value rows
