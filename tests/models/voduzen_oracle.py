@@ -191,3 +191,11 @@ def random_weights(cfg, seed=0):
                 W[p + "shared.up"], W[p + "shared.down"] = rnd(f["shared"]["ff"], n, gain=1.5), rnd(n, f["shared"]["ff"])
                 W[p + "shared.sg"] = rnd(1, n, gain=1.5)
     return W
+
+
+def greedy(cfg, W, prompt, n):
+    """The ``n`` tokens that greedy decoding appends."""
+    toks = list(prompt)
+    for _ in range(n):
+        toks.append(int(forward(W, cfg, toks)[-1].argmax()))
+    return toks[len(prompt):]
