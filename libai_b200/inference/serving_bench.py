@@ -2,7 +2,9 @@
 attention with chunk / kept-first window masks and mixture-of-experts feed-forwards) beside Llama at equal width, depth and
 (active) feed-forward size, and of Salizen (hyper-connection streams, linear-attention recurrences, sink-softmax window
 attention) beside Nefelorn, and of Zubarax (post-norm blocks, paged attention with mixed heads beside an HGRN2 recurrence,
-input-weighted experts) beside Salizen, random weights, one GPU.  ``bench.py --serving [--serving-model nefelorn|salizen|zubarax]`` prints the result
+input-weighted experts) beside Salizen, and of Voduzen (latent attention over the whole past, norms on the sublayers' outputs,
+experts that may pass a token on) beside Bumodra and Zubarax, random weights, one GPU.
+``bench.py --serving [--serving-model nefelorn|salizen|zubarax|voduzen]`` prints the result
 as one JSON line; ``--serving-kernels`` adds device times of the individual kernels of one block at the same sizes with their
 roofline fractions.
 
@@ -735,11 +737,186 @@ def kernel_table_zubarax(s, batch, prompt):
     return {"peaks": src, "hbm_bytes_per_s": hbm, "bf16_flops": flops, "rows": rows}
 
 
+# ======================================================================================================================
+# Voduzen beside Bumodra (latent attention, dense feed-forward) and Zubarax (paged attention, experts)
+# ======================================================================================================================
+VODUZEN_SIZES = {
+    "w1024": dict(width=1024, heads=8, kv_heads=8, dim=128, rot_dim=64, q_rank=512, kv_rank=256, experts=16, identity=2, top=2, expert_ff=1408,
+                  blocks=4, vocab=32000),
+    "w2048": dict(width=2048, heads=16, kv_heads=16, dim=128, rot_dim=64, q_rank=768, kv_rank=512, experts=32, identity=2, top=2, expert_ff=2816,
+                  blocks=4, vocab=32000),
+}
+
+
+def voduzen_config(s):
+    """Blocks alternate between the two mixers; ``top`` of the experts (or identity experts) and a shared expert of one expert's size."""
+    D, R = s["dim"], s["rot_dim"]
+    moe = {"kind": "moe", "expert": {"ff": s["expert_ff"]}, "router": {"experts": s["experts"], "top": s["top"], "identity": s["identity"]},
+           "shared": {"ff": s["expert_ff"]}}
+    mix = {"heads": s["heads"], "dim": D, "rot_dim": R, "vdim": D, "kv_rank": s["kv_rank"], "scale": (D + R) ** -0.5}
+    direct = dict(mix, rot={"dims": R, "base": 1000000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 24.0, "slow": 2.0}})
+    latent = dict(mix, q_rank=s["q_rank"], rot={"dims": R, "base": 10000.0})
+    layers = [{"type": "latent_attention_2", "mixer": latent, "mlp": moe} if i % 2 else {"type": "latent_attention", "mixer": direct, "mlp": moe}
+              for i in range(s["blocks"])]
+    return dict(vocab=s["vocab"], width=s["width"], norm={"eps": 1e-6}, embedding={"scale": s["width"] ** 0.5}, logit_scale=1.0, layers=layers)
+
+
+def bumodra_latent_config(s, prompt):
+    """Bumodra with every block a latent-attention one whose window covers the prompt and the decoded tokens, the same latents and heads
+    (no rotated part), and a dense feed-forward of the active experts' size."""
+    att = {"type": "latent_attention", "mlp": {"kind": "dense", "ff": (s["top"] + 1) * s["expert_ff"]},
+           "mixer": {"heads": s["heads"], "dim": s["dim"], "vdim": s["dim"], "q_rank": s["q_rank"], "kv_rank": s["kv_rank"],
+                     "mask": {"size": prompt + 64}, "scale": s["dim"] ** -0.5}}
+    return dict(vocab=s["vocab"], width=s["width"], norm={"eps": 1e-6}, layers=[att for _ in range(s["blocks"])])
+
+
+@torch.no_grad()
+def throughput_voduzen(s, batch, prompt, new_tokens, steps, warmup):
+    from libai_b200.config import DictConfig
+    from libai_b200.layers._param import param_defaults
+    from libai_b200.models import BumodraForCausalLM, VoduzenForCausalLM, ZubaraxForCausalLM
+
+    ids = torch.randint(1, s["vocab"], (batch, prompt), generator=torch.Generator().manual_seed(0))
+    out = {}
+    for name, cls, cfg in (("voduzen", VoduzenForCausalLM, voduzen_config(s)), ("bumodra", BumodraForCausalLM, bumodra_latent_config(s, prompt)),
+                           ("zubarax", ZubaraxForCausalLM, zubarax_config(dict(s, kv_heads=s["kv_heads"] // 4)))):
+        with param_defaults(dtype=torch.bfloat16, device="cuda", seed=1):
+            model = cls(DictConfig(cfg)).eval().cuda()
+        _stateful_throughput(model, name, ids, batch, new_tokens, steps, warmup, out)
+        del model
+        torch.cuda.empty_cache()
+    return out
+
+
+@torch.no_grad()
+def kernel_table_voduzen(s, batch, prompt):
+    """Device time of every kernel of a Voduzen block at these sizes (prefill rows = batch·prompt; decode rows = batch) beside the like
+    kernel of Bumodra, Zubarax or Nefelorn, with the bytes / FLOPs the operation needs and the fraction of the measured roofline."""
+    from libai_b200.inference.ragged import RaggedBatch
+    from libai_b200.inference.state_cache import SequenceStateCache
+    from libai_b200.layers import DynamicTanh, MoEFeedForward
+    from libai_b200.layers._param import param_defaults
+    from libai_b200.ops import kv_functional as KF
+    from libai_b200.ops import latent_functional as LF
+    from libai_b200.ops import paged_functional as PF
+    from libai_b200.ops import seq_functional as SF
+
+    hbm, flops, src = _peaks()
+    dev, bf = "cuda", torch.bfloat16
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    n, H, D, R, C, QR = s["width"], s["heads"], s["dim"], s["rot_dim"], s["kv_rank"], s["q_rank"]
+    E, I, top, ff = s["experts"], s["identity"], s["top"], s["expert_ff"]
+    V, CS = D, LF.row_channels(s["kv_rank"], s["rot_dim"])
+    rows = []
+
+    def add(name, fn, bytes_=0.0, fl=0.0):
+        ms = _time(fn, flush=flush)
+        ideal = max(bytes_ / hbm, fl / flops) * 1e3
+        rows.append(dict(kernel=name, ms=round(ms, 4), ideal_ms=round(ideal, 5), roofline_fraction=round(ideal / ms, 4),
+                         bound="memory" if bytes_ / hbm >= fl / flops else "tensor"))
+
+    rnd = lambda *shape: torch.randn(*shape, device=dev).to(bf)
+    with param_defaults(dtype=bf, device=dev, seed=2):
+        na, nb = DynamicTanh(n), DynamicTanh(n)
+        moe = MoEFeedForward(n, ff, E, top, router="softmax_all", act="relu2", identity=I, correction=True, gated=False)
+        zmoe = MoEFeedForward(n, ff, E, top, router="sigmoid_raw", act="swish_clamp", limit=7.0, weight_input=True)
+    cache = SequenceStateCache(dev, bf, max_slots=batch, page_size=64)
+    handle = cache.register("paged", channels=CS, taps=1, conv_channels=0)
+    slots = cache.allocate(batch)
+    cache.prepare(slots, [prompt + 1] * batch)
+    bufs = cache.buffers(handle)
+    pool, table = bufs["pool"], bufs["table"]
+    pool.copy_(rnd(*pool.shape))
+    freq = KF.rotary_frequencies(R, 1e4)[0].to(dev)
+    uk, uv, ukv, uq = rnd(H * D, C), rnd(H * V, C), rnd(H * (D + V), C), rnd(H * (D + R), QR)
+    sink = torch.zeros(H, device=dev)
+    w, wc, wqn = torch.zeros(n, dtype=bf, device=dev), torch.ones(C, dtype=bf, device=dev), torch.ones(QR, dtype=bf, device=dev)
+    for phase, lens, past in (("prefill", [prompt] * batch, [0] * batch), ("decode", [1] * batch, [prompt] * batch)):
+        rb = RaggedBatch(lens, slots, past, dev)
+        T = rb.tokens
+        x, y32, h = torch.randn(T, n, device=dev), torch.randn(T, n, device=dev), torch.empty(T, n, dtype=bf, device=dev)
+        add(f"{phase}: outer-norm residual (x + RMS norm(y), fp32 residual + bf16 copy)", lambda: PF.outnorm_residual(x, w, 1e-6, y=y32, h=h), T * n * 14)
+        add(f"{phase}: Zubarax post-norm residual", lambda: PF.postnorm_residual(x, w, 1e-6, alpha=2.0, y=y32, h=h), T * n * 14)
+        add(f"{phase}: Nefelorn closing norm + residual + opening norm", lambda: KF.dyt_residual(x, y32, post=na.triple(), nxt=nb.triple(), h=h), T * n * 14)
+        proj = rnd(T, QR + C + R)
+        dq, dkv = proj[:, :QR], proj[:, QR:]
+        cq, c = torch.empty(T, QR, dtype=bf, device=dev), torch.empty(T, C, dtype=bf, device=dev)
+        packed = phase == "prefill"
+        add(f"{phase}: latent norms + rotation + page write", lambda: LF.latent_prepare(dkv, wc, freq, 1.0, 1e-6, pool, table, rb, C, R, dq=dq, wq=wqn, packed=packed),
+            T * ((QR + C + R) * 2 + QR * 2 + CS * 2 * (2 if packed else 1) + R * 4))
+
+        def bumodra_norms():
+            SF.rms_norm_rows(dq, wqn, offset=0.0, eps=1e-6, out=cq)
+            SF.rms_norm_rows(dkv[:, :C], wc, offset=0.0, eps=1e-6, out=c)
+
+        ring = rnd(batch, prompt + 64, C)
+        add(f"{phase}: Bumodra latent norms (two kernels)", bumodra_norms, T * (QR + C) * 4)
+        add(f"{phase}: Bumodra latent ring write", lambda: SF.latent_write(ring, c, rb), T * C * 4)
+        q = rnd(T, H * (D + R))
+        cs, _, lat = LF.latent_prepare(dkv, wc, freq, 1.0, 1e-6, pool, table, rb, C, R, packed=True)
+        yb = torch.empty(T, H * V, dtype=bf, device=dev)
+        sc = (D + R) ** -0.5
+        if phase == "prefill":
+            pairs = prompt * (prompt + 1) // 2 * batch
+            kv = rnd(T, H * (D + V))
+            add("prefill: key/value expansion of the latents (tcgen05 GEMM)", lambda: KF.linear(lat[:, :C], ukv), 0.0, T * C * H * (D + V) * 2.0)
+            add("prefill: latent attention, expanded, rotated part + sink (mma.m16n8k16)",
+                lambda: LF.latent_prompt(q, kv, lat, rb.seq_off, cs, rb, yb, H, D, R, V, C, sc, sink=sink),
+                T * (H * (2 * D + R + 2 * V) + R) * 2, pairs * H * (D + R + V) * 2.0)
+            qd = q[:, :H * D].contiguous()
+            add("prefill: Bumodra window attention, window = prompt (mma.m16n8k16, no rotated part)",
+                lambda: SF.window_attention(qd, kv, None, rb, yb, H, D, V, prompt + 64, sc), T * H * (2 * D + 2 * V) * 2, pairs * H * (D + V) * 2.0)
+        else:
+            live = batch * (prompt + 1)
+            add("decode: absorbed attention over the pages (absorb, mma.m16n8k16, merge + value up-projection)",
+                lambda: LF.latent_absorbed(q, uk, uv, cs, pool, table, rb, yb, H, D, R, V, C, sc, sink=sink), live * CS * 2 + (uk.numel() + uv.numel()) * 2)
+            uk3, uv3, qd = uk.view(H, D, C), uv.view(H, V, C), q[:, :H * D].contiguous()
+
+            def bumodra_decode():
+                qa = torch.einsum("bhd,hdc->bhc", qd.view(T, H, D).float(), uk3.float())
+                la = SF.latent_decode(qa.contiguous(), ring, c, rb, prompt + 64, sc)
+                SF.head_gate(torch.einsum("bhc,hvc->bhv", la, uv3.float()).contiguous(), None, yb, H, V)
+
+            add("decode: Bumodra absorbed attention over its ring (einsum, kernel, einsum, gate)", bumodra_decode, live * C * 2 + (uk.numel() + uv.numel()) * 2)
+            qa = torch.randn(batch, H, C, device=dev)
+            add("decode: Bumodra absorbed attention, its kernel alone", lambda: SF.latent_decode(qa, ring, c, rb, prompt + 64, sc), live * C * 2)
+        hb = rnd(T, n)
+        wr = rnd(-(-(E + I + 1) // 8) * 8, n)
+        add(f"{phase}: router (softmax over {E} + {I}, corrected choice, top-{top}) with the token gate's logit",
+            lambda: KF.moe_route(hb, None, top, 1.0, mode=KF.ROUTE_SOFTMAX_ALL, z=KF.router_logits(hb, wr), choices=E + I, experts=E), T * n * 2 + wr.numel() * 2)
+        add(f"{phase}: Zubarax router (sigmoid scores as they are)", lambda: KF.moe_route(hb, zmoe.router, top, 1.0, mode=KF.ROUTE_SIGMOID_RAW), T * n * 2 + E * n * 2)
+        act_rows = int(T * top * E / (E + I))
+        add(f"{phase}: routed experts (route, sort, W_up, relu^2, W_down)", lambda: moe.run(hb, graph_safe=rb.single), min(E, act_rows) * 2 * ff * n * 2 + T * n * 6,
+            act_rows * 2 * ff * n * 2.0)
+        add(f"{phase}: Zubarax routed experts (gated)", lambda: zmoe.run(hb, graph_safe=rb.single), min(E, T * top) * 3 * ff * n * 2 + T * n * 6, T * top * 3 * ff * n * 2.0)
+        r, zr, gate = moe.run(hb, graph_safe=rb.single), zmoe.run(hb, graph_safe=rb.single), torch.randn(T, device=dev)
+        moved = T * n * 14 + (T * n * 4 * top if r.pos is not None else T * n * 4)
+        add(f"{phase}: outer-norm residual with gated shared expert, routed rows and identity share",
+            lambda: PF.outnorm_residual(x, w, 1e-6, y=y32, gate=gate, y2=r.y, pos=r.pos, cw=r.wts, keep=r.keep, h=h), moved)
+        add(f"{phase}: Zubarax post-norm residual with shared expert and routed rows",
+            lambda: PF.postnorm_residual(x, w, 1e-6, alpha=2.0, y=y32, y2=zr.y, pos=zr.pos, h=h), moved)
+    return {"peaks": src, "hbm_bytes_per_s": hbm, "bf16_flops": flops, "rows": rows}
+
+
 def main(args):
     assert torch.cuda.is_available(), "the serving bench needs a GPU"
     from libai_b200 import ops
 
     ops.reset_launch_count()
+    if getattr(args, "serving_model", "bumodra") == "voduzen":
+        result = {"metric": "prefill / decode tokens per second, Voduzen beside Bumodra (latent attention, window = prompt, dense feed-forward of the active size) and Zubarax (paged attention, experts) at equal width, depth and heads",
+                  "dtype": "bf16", "data": "synthetic tokens, random-init weights", "n_gpus": 1, "sizes": {}}
+        for name in (args.serving_sizes.split(",") if args.serving_sizes else list(VODUZEN_SIZES)):
+            s = VODUZEN_SIZES[name]
+            r = throughput_voduzen(s, args.serving_batch, args.serving_prompt, new_tokens=max(args.steps, 8),
+                                   steps=max(args.steps // 2, 3), warmup=max(args.warmup, 3))
+            if args.serving_kernels:
+                r["kernels"] = kernel_table_voduzen(s, args.serving_batch, args.serving_prompt)
+            result["sizes"][name] = {"config": dict(s), "batch": args.serving_batch, "prompt": args.serving_prompt, **r}
+            torch.cuda.empty_cache()
+        result["gpu_launches"] = ops.launch_count()
+        print(json.dumps(result))
+        return
     if getattr(args, "serving_model", "bumodra") == "zubarax":
         result = {"metric": "prefill / decode tokens per second, Zubarax beside Salizen (window = prompt, one stream) at equal width, depth, heads and expert sizes",
                   "dtype": "bf16", "data": "synthetic tokens, random-init weights", "n_gpus": 1, "sizes": {}}
