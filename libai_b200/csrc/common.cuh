@@ -225,8 +225,8 @@ LB_DEVICE void tmem_dealloc_2cta(uint32_t taddr) {
   asm volatile("tcgen05.dealloc.cta_group::2.sync.aligned.b32 %0, %1;\n" ::"r"(taddr), "n"(kCols) : "memory");
 }
 // arrive (count 1) on the mbarrier at the same shared-memory offset in CTA `cta` of the cluster (the form CUTLASS'
-// ClusterBarrier::arrive(cta_id) uses; an explicit `.release.cluster` compiles to MEMBAR.ALL.GPU + ERRBAR per arrival,
-// which throttled the peer's TMA producer to one k-block per fence: profiles/r2_10_ncu_gemm_2cta_first.txt)
+// ClusterBarrier::arrive(cta_id) uses; with an explicit `.release.cluster` per arrival the peer's TMA producer was measured
+// throttled to one k-block per arrival: profiles/r2_10_ncu_gemm_2cta_first.txt)
 LB_DEVICE void mbar_arrive_cluster(uint64_t* bar, uint32_t cta) {
   asm volatile(
       "{\n\t.reg .b32 ra;\n\t"
@@ -373,17 +373,16 @@ LB_DEVICE uint32_t pack_bf16(float a, float b) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 LB_DEVICE float2 unpack_bf16(uint32_t u) {
-  // a bf16 is the upper half of an fp32: one shift for the low element, one mask for the high one (the intrinsic
-  // compiled to PRMT + IMAD for the high half)
+  // a bf16 is the upper half of an fp32: one shift for the low element, one mask for the high one
   return make_float2(__uint_as_float(u << 16), __uint_as_float(u & 0xffff0000u));
 }
 
 enum Act : int { ACT_NONE = 0, ACT_GELU = 1, ACT_GELU_TANH = 2, ACT_RELU = 3, ACT_SILU = 4, ACT_QUICK_GELU = 5,
                  ACT_RESADD = 6 /* GEMM epilogue only: out = acc (+ bias) + pre_in, i.e. the residual add */ };
 
-// erfc(|x|/sqrt2) and exp(-x^2/2) from one MUFU.EX2 + one MUFU.RCP (Abramowitz-Stegun 7.1.26, |err(erf)| < 1.5e-7 -
-// three orders of magnitude below bf16 resolution).  The libm erff costs ~60 instructions with a divergent branch,
-// which made the 4-warp GEMM epilogue (one thread per accumulator row) the bottleneck of the h->4h projection.
+// erfc(|x|/sqrt2) and exp(-x^2/2) from one ex2.approx and one rcp.approx (Abramowitz-Stegun 7.1.26, |err(erf)| < 1.5e-7 -
+// three orders of magnitude below bf16 resolution).  With erff() the 4-warp GEMM epilogue (one thread per accumulator row)
+// was measured to be the bottleneck of the h->4h projection.
 LB_DEVICE void gelu_terms(float x, float& erfc_abs, float& gauss) {
   const float z = fabsf(x) * 0.70710678118654752f;
   float t;
@@ -410,8 +409,7 @@ LB_DEVICE float gelu_grad_fast(float x) {
   const float cdf = x >= 0.f ? 1.0f - h : h;
   return fmaf(x * 0.3989422804014327f, e, cdf);
 }
-// 2^x on the SFU without the denormal-range fix-up branch that exp2f() compiles to (one BSSY/BRA/BSYNC triple per
-// element in the softmax loops); ex2.approx(-inf) = +0.
+// 2^x through ex2.approx (measured faster than exp2f() in the softmax loops); ex2.approx(-inf) = +0.
 LB_DEVICE float fast_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
