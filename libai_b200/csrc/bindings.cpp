@@ -75,6 +75,9 @@ struct LbRngArgs {
   int captured;
   unsigned long long salt;
 };
+int lb_latent_prompt_tc(const void* q, long ldq, const void* kv, long ldkv, const void* rot, long ldr, const float* cs, const float* sink,
+                        const int* ext_off, const int* qt_seq, const int* qt_start, int ntiles, const int* seq_off, const int* past, void* y,
+                        long ldy, long tokens, long rows, int H, int D, int R, int V, float scale, int* err, cudaStream_t s);
 int lb_attn_fwd(const void* q, const void* k, const void* v, void* o, float* lse, int B, int A, int S, int D,
                 const long* q_strides, const long* k_strides, const long* v_strides, int causal, float scale,
                 const int* kv_lens, const void* bias, const long* bias_strides, const float* alibi_slopes, float p_drop,
@@ -167,6 +170,39 @@ void gemm_grouped(const Tensor& a, const Tensor& w, const std::vector<int64_t>& 
                        (int)out.stride(0), 0, epi, nullptr, 0, nullptr, 0, 0, cur_stream()), "gemm_grouped");
     at += c;
   }
+}
+
+// Causal attention of ragged prompts on expanded latents (csrc/latent_attention_sm100.cu): q [tokens, H*(D+R)] with the R part
+// unrotated, kv [rows, H*D | H*V], rot [rows, R] the shared rotated key part, cs [tokens, R/2, 2]; query tiles of 128
+void latent_prompt_tc(const Tensor& q, const Tensor& kv, const Tensor& rot, const Tensor& cs, const c10::optional<Tensor>& sink, const Tensor& ext_off,
+                      const Tensor& seq_off, const Tensor& past, const Tensor& qt_seq, const Tensor& qt_start, Tensor y, int64_t H, int64_t D,
+                      int64_t R, int64_t V, double scale) {
+  for (const Tensor* t : {&q, &kv, &rot, (const Tensor*)&y})
+    TORCH_CHECK(t->is_cuda() && t->dim() == 2 && t->stride(1) == 1 && t->scalar_type() == at::kBFloat16, "latent_prompt_tc: bf16 row-major matrices expected");
+  TORCH_CHECK(q.size(1) == H * (D + R) && kv.size(1) == H * (D + V) && rot.size(1) == R && rot.size(0) == kv.size(0) && y.size(0) == q.size(0) &&
+              y.size(1) == H * V && scale > 0, "latent_prompt_tc: shapes");
+  TORCH_CHECK(cs.is_cuda() && cs.scalar_type() == at::kFloat && cs.is_contiguous() && cs.numel() == q.size(0) * R, "latent_prompt_tc: cs fp32 [tokens, R/2, 2]");
+  for (const Tensor* t : {&ext_off, &seq_off, &past, &qt_seq, &qt_start})
+    TORCH_CHECK(t->is_cuda() && t->scalar_type() == at::kInt && t->is_contiguous(), "latent_prompt_tc: int32 CUDA metadata expected");
+  TORCH_CHECK(qt_seq.numel() == qt_start.numel() && ext_off.numel() == seq_off.numel() && past.numel() + 1 == seq_off.numel(), "latent_prompt_tc: metadata sizes");
+  const float* sp = nullptr;
+  if (sink.has_value() && sink->defined()) {
+    TORCH_CHECK(sink->is_cuda() && sink->scalar_type() == at::kFloat && sink->is_contiguous() && sink->numel() == H, "latent_prompt_tc: sink fp32 [H]");
+    sp = sink->data_ptr<float>();
+  }
+  static int* err = nullptr;                     // mapped host word: a kernel whose bounded wait ran out sets it
+  if (err == nullptr) {
+    TORCH_CHECK(cudaHostAlloc(reinterpret_cast<void**>(&err), sizeof(int), cudaHostAllocMapped) == cudaSuccess, "latent_prompt_tc: mapped host word");
+    *err = 0;
+  }
+  TORCH_CHECK(*static_cast<volatile int*>(err) == 0, "latent_prompt_tc: a wait ran out in an earlier launch; its result is invalid");
+  int* err_dev = nullptr;
+  TORCH_CHECK(cudaHostGetDevicePointer(reinterpret_cast<void**>(&err_dev), err, 0) == cudaSuccess, "latent_prompt_tc: mapped host word");
+  c10::cuda::CUDAGuard guard(q.device());
+  check(lb_latent_prompt_tc(q.data_ptr(), q.stride(0), kv.data_ptr(), kv.stride(0), rot.data_ptr(), rot.stride(0), cs.data_ptr<float>(), sp,
+                            ext_off.data_ptr<int>(), qt_seq.data_ptr<int>(), qt_start.data_ptr<int>(), (int)qt_seq.numel(), seq_off.data_ptr<int>(),
+                            past.data_ptr<int>(), y.data_ptr(), y.stride(0), q.size(0), kv.size(0), (int)H, (int)D, (int)R, (int)V, (float)scale, err_dev,
+                            cur_stream()), "latent_prompt_tc");
 }
 
 // The same as ONE launch with the groups known on the device only: `a` [M, K] with M a multiple of 128, every 128-row block
@@ -835,6 +871,7 @@ TORCH_LIBRARY(libai_b200, m) {
   m.def("gemm(Tensor a, Tensor b, int layout, Tensor? bias, Tensor? out, bool accumulate, ScalarType out_dtype) -> Tensor", &gemm);
   m.def("gemm_grouped(Tensor a, Tensor w, int[] counts, Tensor(a!) out) -> ()", &gemm_grouped);
   m.def("gemm_grouped_blocks(Tensor a, Tensor w, Tensor tile_group, Tensor(a!) out) -> ()", &gemm_grouped_blocks);
+  m.def("latent_prompt_tc(Tensor q, Tensor kv, Tensor rot, Tensor cs, Tensor? sink, Tensor ext_off, Tensor seq_off, Tensor past, Tensor qt_seq, Tensor qt_start, Tensor(a!) y, int H, int D, int R, int V, float scale) -> ()", &latent_prompt_tc);
   m.def("linear_bias_residual(Tensor x, Tensor w, Tensor? bias, Tensor residual) -> Tensor", &linear_bias_residual);
   m.def("embedding_fwd(Tensor ids, Tensor table, int vocab_start) -> Tensor", &embedding_fwd);
   m.def("embedding_bwd(Tensor ids, Tensor gy, Tensor(a!) grad, int vocab_start) -> ()", &embedding_bwd);

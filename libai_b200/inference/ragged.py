@@ -96,7 +96,7 @@ class RaggedBatch:
         self._ext: Dict[int, WindowExt] = {}
         self._kv_ext: Dict[tuple, KvExt] = {}
         self._page_ext = None
-        self._tiles: Dict[int, tuple] = {}
+        self._tiles: Dict[tuple, tuple] = {}
 
     def ext(self, window: int) -> WindowExt:
         if window not in self._ext:
@@ -115,14 +115,17 @@ class RaggedBatch:
             self._page_ext = PageExt(self)
         return self._page_ext
 
-    def query_tiles(self, size: int):
-        """Tiles of ``size`` consecutive new tokens of one sequence: (sequence of every tile, its first token) on the device."""
-        if size not in self._tiles:
-            seq = [b for b, n in enumerate(self.lens) for _ in range(0, n, size)]
-            start = [t for n in self.lens for t in range(0, n, size)]
-            packed = torch.tensor(seq + start, dtype=torch.int32).to(self.device, non_blocking=True)
-            self._tiles[size] = (packed[: len(seq)], packed[len(seq):])
-        return self._tiles[size]
+    def query_tiles(self, size: int, longest_first: bool = False):
+        """Tiles of ``size`` consecutive new tokens of one sequence: (sequence of every tile, its first token) on the device;
+        ``longest_first``: in the order of falling positions (under a causal mask the late tiles have the most keys)."""
+        key = (size, longest_first)
+        if key not in self._tiles:
+            tiles = [(b, t) for b, n in enumerate(self.lens) for t in range(0, n, size)]
+            if longest_first:
+                tiles.sort(key=lambda bt: -(self.past_list[bt[0]] + bt[1]))
+            packed = torch.tensor([b for b, _ in tiles] + [t for _, t in tiles], dtype=torch.int32).to(self.device, non_blocking=True)
+            self._tiles[key] = (packed[: len(tiles)], packed[len(tiles):])
+        return self._tiles[key]
 
     def last_rows(self) -> List[int]:
         """Packed row of every sequence's last new token."""

@@ -796,6 +796,7 @@ def kernel_table_voduzen(s, batch, prompt):
     from libai_b200.inference.state_cache import SequenceStateCache
     from libai_b200.layers import DynamicTanh, MoEFeedForward
     from libai_b200.layers._param import param_defaults
+    from libai_b200.ops import functional as OF
     from libai_b200.ops import kv_functional as KF
     from libai_b200.ops import latent_functional as LF
     from libai_b200.ops import paged_functional as PF
@@ -860,9 +861,13 @@ def kernel_table_voduzen(s, batch, prompt):
             pairs = prompt * (prompt + 1) // 2 * batch
             kv = rnd(T, H * (D + V))
             add("prefill: key/value expansion of the latents (tcgen05 GEMM)", lambda: KF.linear(lat[:, :C], ukv), 0.0, T * C * H * (D + V) * 2.0)
-            add("prefill: latent attention, expanded, rotated part + sink (mma.m16n8k16)",
-                lambda: LF.latent_prompt(q, kv, lat, rb.seq_off, cs, rb, yb, H, D, R, V, C, sc, sink=sink),
-                T * (H * (2 * D + R + 2 * V) + R) * 2, pairs * H * (D + R + V) * 2.0)
+            for name, tc in (("tcgen05", True), ("mma.m16n8k16, for other head sizes", False)):
+                add(f"prefill: latent attention, expanded, rotated part + sink ({name})",
+                    lambda: LF.latent_prompt(q, kv, lat, rb.seq_off, cs, rb, yb, H, D, R, V, C, sc, sink=sink, tc=tc),
+                    T * (H * (2 * D + R + 2 * V) + R) * 2, pairs * H * (D + R + V) * 2.0)
+            qkv4 = rnd(batch, prompt, H, 3 * D)
+            add("prefill: Llama causal flash attention, same heads (tcgen05, no rotated part)",
+                lambda: OF.attention_qkvpacked(qkv4, causal=True, scale=D ** -0.5), qkv4.numel() * 2 + T * H * D * 2, pairs * H * D * 4.0)
             qd = q[:, :H * D].contiguous()
             add("prefill: Bumodra window attention, window = prompt (mma.m16n8k16, no rotated part)",
                 lambda: SF.window_attention(qd, kv, None, rb, yb, H, D, V, prompt + 64, sc), T * H * (2 * D + 2 * V) * 2, pairs * H * (D + V) * 2.0)

@@ -13,7 +13,7 @@ from typing import Optional
 
 import torch
 
-from . import count_launch, impl, load_kv_ext
+from . import count_launch, impl, load_ext, load_kv_ext
 
 
 def _native(t: torch.Tensor) -> bool:
@@ -92,7 +92,15 @@ def latent_rows(pool, table, rb, lat):
     return torch.cat(parts), ext.ext_off
 
 
-MMA_QUERY_TILE = 64            # queries per block of the tensor-core prompt kernel
+MMA_QUERY_TILE = 64            # queries per block of the mma.sync prompt kernel
+TC_QUERY_TILE = 128            # queries per block of the tcgen05 prompt kernel
+TC_MIN_TOKENS = 64             # a step whose longest sequence brings fewer tokens would leave most of its tile empty
+
+
+def prompt_tc_eligible(q, kv, lat, y, D: int, R: int, V: int, C: int, scale: float) -> bool:
+    """bf16 prompt steps whose sizes the tcgen05 prompt kernel is built for."""
+    return (q.dtype == torch.bfloat16 and D in (64, 128) and V in (64, 128) and R % 8 == 0 and 8 <= R <= 64 and C % 8 == 0 and scale > 0
+            and all(t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 for t in (q, kv, lat, y)))
 
 
 def prompt_mma_eligible(q, kv, lat, y, D: int, R: int, V: int, C: int) -> bool:
@@ -110,13 +118,23 @@ def _softmax_rows(s, sink):
     return torch.softmax(torch.cat([s, extra], -1), -1)[..., :-1]
 
 
-def latent_prompt(q, kv, lat, ext_off, cs, rb, y, H: int, D: int, R: int, V: int, C: int, scale: float, *, sink=None, mma: bool = True):
+def latent_prompt(q, kv, lat, ext_off, cs, rb, y, H: int, D: int, R: int, V: int, C: int, scale: float, *, sink=None, mma: bool = True,
+                  tc: Optional[bool] = None):
     """Causal softmax attention of every packed query over the rows ``0 … its own position`` of its sequence.  ``q``
     ``[tokens, H·(D+R)]`` (per head ``[D | R]``, the ``R`` part still unrotated: it is turned by ``cs``), ``kv`` ``[rows, H·D keys | H·V
     values]`` and the shared rotated key part in columns ``C … C+R`` of ``lat`` ``[rows, row size]``, both laid out by ``ext_off``.
-    ``sink`` (fp32 ``[H]``): the denominator also holds ``exp(sink_h)``.  The result goes to ``y`` ``[tokens, H·V]``.  bf16 inputs whose
-    sizes it is built for take the tensor-core kernel; ``mma=False`` keeps them on the generic one (fp32 inputs always are)."""
+    ``sink`` (fp32 ``[H]``): the denominator also holds ``exp(sink_h)``.  The result goes to ``y`` ``[tokens, H·V]``.  bf16 inputs take the
+    tcgen05 kernel where it is built for their sizes and the step is long enough (``tc`` decides otherwise), then the mma.sync kernel
+    where that one is; ``mma=False`` keeps them on the generic kernel (fp32 inputs always are)."""
     if _native(q):
+        if tc is None:
+            tc = mma and max(rb.lens) >= TC_MIN_TOKENS
+        if tc and prompt_tc_eligible(q, kv, lat, y, D, R, V, C, scale):
+            seq, start = rb.query_tiles(TC_QUERY_TILE, longest_first=True)
+            if seq.numel() <= 65535:
+                count_launch()
+                load_ext(required=True).latent_prompt_tc(q, kv, lat[:, C:C + R], cs, sink, ext_off, rb.seq_off, rb.past, seq, start, y, H, D, R, V, float(scale))
+                return y
         tiles = rb.query_tiles(MMA_QUERY_TILE) if mma and prompt_mma_eligible(q, kv, lat, y, D, R, V, C) else (None, None)
         count_launch()
         load_kv_ext().latent_prompt(q, kv, lat, cs, sink, ext_off, rb.tok_seq, rb.seq_off, rb.past, tiles[0], tiles[1], y, H, D, R, V, C, float(scale))

@@ -612,10 +612,62 @@ def test_every_form_of_the_attention_agrees(H, D, R, V, C, sink):
                  for parts in (1, 3, 40, None) for mma in ((False, True) if dtype == torch.bfloat16 else (False,))}
         if dtype == torch.bfloat16:
             assert LF.prompt_mma_eligible(q, kv, lat, want.to(dtype), D, R, V, C)
-            forms["prompt mma"] = LF.latent_prompt(q, kv, lat, off, cs, rb, new(), *args, sink=sk)
+            forms["prompt mma"] = LF.latent_prompt(q, kv, lat, off, cs, rb, new(), *args, sink=sk, tc=False)
         for name, got in forms.items():
             assert torch.allclose(got.float(), want, atol=tol, rtol=tol), (name, dtype, float((got.float() - want).abs().max()))
             assert float((got.float() - want).abs().mean()) < tol / 8, name
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("H,D,R,V,C", [(3, 64, 16, 64, 40), (2, 64, 64, 128, 96), (4, 128, 24, 64, 72), (5, 128, 64, 128, 256), (1, 64, 8, 64, 16)])
+@pytest.mark.parametrize("gain", [1.0, 8.0])
+def test_tcgen05_prompts_match_the_generic_kernel(H, D, R, V, C, gain):
+    """bf16 prompts on the tcgen05 kernel: several key tiles, tiles that end inside a sequence, continued sequences, a sequence of one
+    token, scores that grow along the sequence so that running maxima move, with and without a sink."""
+    torch.manual_seed(1)
+    lens, past = [300, 1, 129, 128, 70], [0, 250, 383, 0, 61]
+    T = sum(lens)
+    pool, table, rb = cached_rows(torch.bfloat16, lens, past, C, R)
+    lat, off = LF.latent_rows(pool, table, rb, None)
+    kv = torch.randn(lat.shape[0], H * (D + V), device="cuda")
+    kv[:, :H * D] *= torch.linspace(0.2, 1.5, lat.shape[0], device="cuda")[:, None]
+    kv = kv.to(torch.bfloat16)
+    q = (gain * torch.randn(T, H * (D + R), device="cuda")).to(torch.bfloat16)
+    ang = torch.rand(T, R // 2, device="cuda") * 6
+    cs = torch.stack([ang.cos(), ang.sin()], -1).contiguous()
+    if gain > 1:                                                    # large scores: quarter turns, so that no kernel rounds a rotated query
+        cs = cs.round().where(cs.abs() == cs.abs().amax(-1, keepdim=True), torch.zeros_like(cs)).sign().contiguous()
+    for sk in (None, torch.randn(H, device="cuda") + 2):
+        args = (H, D, R, V, C, (D + R) ** -0.5)
+        new = lambda: torch.full((T, H * V), float("nan"), device="cuda", dtype=torch.bfloat16)
+        want = LF.latent_prompt(q, kv, lat, off, cs, rb, new(), *args, sink=sk, mma=False).float()
+        assert LF.prompt_tc_eligible(q, kv, lat, new(), D, R, V, C, 0.1)
+        got = LF.latent_prompt(q, kv, lat, off, cs, rb, new(), *args, sink=sk, tc=True).float()
+        other = LF.latent_prompt(q, kv, lat, off, cs, rb, new(), *args, sink=sk, tc=False).float()
+        for name, g in (("tcgen05", got), ("mma.sync", other)):
+            assert torch.allclose(g, want, atol=3e-2, rtol=3e-2), (name, float((g - want).abs().max()))
+            assert float((g - want).abs().mean()) < 3e-3, name
+        assert not torch.equal(got, other)                          # the two did run different kernels
+
+
+@pytest.mark.gpu
+def test_bf16_model_on_the_tcgen05_path(tmp_path, monkeypatch):
+    """A whole bf16 model whose sizes the tcgen05 prompt kernel takes: against the oracle, and against the same model kept off it."""
+    cfg = O.model_cfg([O.layer(O.mixer_cfg(heads=2, dim=64, rot_dim=16, vdim=64, kv_rank=40, scale=0.11, scaling=YARN)),
+                       O.layer(O.mixer_cfg(heads=3, dim=64, rot_dim=32, vdim=64, kv_rank=48, q_rank=40, scale=0.1))], width=64)
+    W = O.random_weights(cfg, seed=5)
+    model = load_pretrained(save_model(tmp_path, cfg, W), dtype=torch.bfloat16, device="cuda")
+    model.kv_page_size = 16
+    prompts = [tokens(170, seed=1), tokens(33, seed=2)]
+    want = [O.forward(W, cfg, p) for p in prompts]
+    cuts = [[140, 20] + [1] * 10, [33]]
+    fast = run_schedule(model, prompts, cuts)
+    monkeypatch.setattr(LF, "prompt_tc_eligible", lambda *a: False)
+    slow = run_schedule(model, prompts, cuts)
+    for f, s_, w in zip(fast, slow, want):
+        assert rel_err(f, w) < 1e-1 and rel_err(s_, w) < 1e-1
+        assert rel_err(f, s_.float().cpu()) < 5e-2
+    assert not torch.equal(fast[0], slow[0])                       # the two paths did run different kernels
 
 
 @pytest.mark.gpu
