@@ -52,42 +52,29 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 }
 __device__ __forceinline__ float sigmoidf_(float x) { return 1.f / (1.f + expf(-x)); }
 
-// dot product of a weight row with a vector staged in shared memory as fp32; the lanes of one warp share the row.
+// this lane's share of the products of two weight rows with the same staged vector: both rows' loads are in flight together (the
+// second row may repeat the first).  xs: shared memory, 16-byte aligned when n is a multiple of 16 bytes' worth of T
 template <typename T>
-__device__ __forceinline__ float warp_dot(const T* __restrict__ w, const float* __restrict__ xs, int n, int lane);
-template <>
-__device__ __forceinline__ float warp_dot<float>(const float* __restrict__ w, const float* __restrict__ xs, int n, int lane) {
-  float acc = 0.f;
-  if ((n & 3) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {
+__device__ __forceinline__ float2 lane_dot2(const T* __restrict__ w0, const T* __restrict__ w1, const float* __restrict__ xs, int n, int lane) {
+  constexpr int PER = 16 / sizeof(T);
+  float2 acc = make_float2(0.f, 0.f);
+  if (n % PER == 0 && ((reinterpret_cast<uintptr_t>(w0) | reinterpret_cast<uintptr_t>(w1)) & 15) == 0) {
 #pragma unroll 4
-    for (int i = lane * 4; i < n; i += 128) {
-      const float4 v = *reinterpret_cast<const float4*>(w + i);
-      acc += v.x * xs[i] + v.y * xs[i + 1] + v.z * xs[i + 2] + v.w * xs[i + 3];
-    }
-  } else {
-    for (int i = lane; i < n; i += 32) acc += w[i] * xs[i];
-  }
-  return warp_sum(acc);
-}
-template <>
-__device__ __forceinline__ float warp_dot<__nv_bfloat16>(const __nv_bfloat16* __restrict__ w, const float* __restrict__ xs, int n,
-                                                         int lane) {
-  float acc = 0.f;
-  if ((n & 7) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {
-#pragma unroll 4
-    for (int i = lane * 8; i < n; i += 256) {
-      const uint4 raw = *reinterpret_cast<const uint4*>(w + i);
-      const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw);
+    for (int i = lane * PER; i < n; i += 32 * PER) {
+      const uint4 r0 = *reinterpret_cast<const uint4*>(w0 + i), r1 = *reinterpret_cast<const uint4*>(w1 + i);
+      const T* p0 = reinterpret_cast<const T*>(&r0);
+      const T* p1 = reinterpret_cast<const T*>(&r1);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float2 f = __bfloat1622float2(p[j]);
-        acc += f.x * xs[i + 2 * j] + f.y * xs[i + 2 * j + 1];
+      for (int j = 0; j < PER; j += 4) {          // the staged vector four numbers at a time
+        const float4 x = *reinterpret_cast<const float4*>(xs + i + j);
+        acc.x += ldf(p0 + j) * x.x + ldf(p0 + j + 1) * x.y + ldf(p0 + j + 2) * x.z + ldf(p0 + j + 3) * x.w;
+        acc.y += ldf(p1 + j) * x.x + ldf(p1 + j + 1) * x.y + ldf(p1 + j + 2) * x.z + ldf(p1 + j + 3) * x.w;
       }
     }
   } else {
-    for (int i = lane; i < n; i += 32) acc += __bfloat162float(w[i]) * xs[i];
+    for (int i = lane; i < n; i += 32) { acc.x += ldf(w0 + i) * xs[i]; acc.y += ldf(w1 + i) * xs[i]; }
   }
-  return warp_sum(acc);
+  return acc;
 }
 
 // ------------------------------------------------------------------------------------------------------------------
@@ -960,7 +947,7 @@ __global__ void __launch_bounds__(256)
 moe_pair_gateup_kernel(const T* __restrict__ h, long ldh, const T* __restrict__ wgu, const int* __restrict__ idx,
                        const float* __restrict__ wts, int win, T* __restrict__ a, int E, int ff, int n, int top, int act, int gated,
                        float limit) {
-  extern __shared__ float sm[];
+  extern __shared__ __align__(16) float sm[];
   const long pair = blockIdx.x;
   const long tok = pair / top;
   const int e = idx[pair];
@@ -976,14 +963,21 @@ moe_pair_gateup_kernel(const T* __restrict__ h, long ldh, const T* __restrict__ 
   const int per = (ff + gridDim.y - 1) / gridDim.y;
   const int f0 = blockIdx.y * per, f1 = min(ff, f0 + per);
   const T* wg = wgu + (long)e * (gated ? 2 : 1) * ff * n;
-  for (int f = f0 + warp; f < f1; f += nw) {
-    if (!gated) {
-      const float v = warp_dot<T>(wg + (long)f * n, sm, n, lane);
-      if (lane == 0) stf(a + pair * ff + f, act_apply(v, act));
-      continue;
+  if (!gated) {                                  // two rows per turn, as the gated form has
+    for (int f = f0 + warp; f < f1; f += 2 * nw) {
+      const int f2 = f + nw < f1 ? f + nw : f;
+      const float2 d = lane_dot2<T>(wg + (long)f * n, wg + (long)f2 * n, sm, n, lane);
+      const float v = warp_sum(d.x), u = warp_sum(d.y);
+      if (lane == 0) {
+        stf(a + pair * ff + f, act_apply(v, act));
+        if (f2 != f) stf(a + pair * ff + f2, act_apply(u, act));
+      }
     }
-    const float gv = warp_dot<T>(wg + (long)f * n, sm, n, lane);
-    const float uv = warp_dot<T>(wg + (long)(ff + f) * n, sm, n, lane);
+    return;
+  }
+  for (int f = f0 + warp; f < f1; f += nw) {
+    const float2 d = lane_dot2<T>(wg + (long)f * n, wg + (long)(ff + f) * n, sm, n, lane);
+    const float gv = warp_sum(d.x), uv = warp_sum(d.y);
     if (lane == 0) stf(a + pair * ff + f, gated_apply(gv, uv, act, limit));
   }
 }
@@ -992,21 +986,33 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 moe_pair_down_kernel(const T* __restrict__ a, const T* __restrict__ wd, const int* __restrict__ idx, const float* __restrict__ wts,
                      int win, float* __restrict__ out, int E, int ff, int n, int top) {
-  extern __shared__ float sm[];
+  extern __shared__ __align__(16) float sm[];
   const long tok = blockIdx.x;
-  for (int i = threadIdx.x; i < top * ff; i += blockDim.x) if (idx[tok * top + i / ff] < E) sm[i] = ldf(a + tok * top * ff + i);
+  for (int k = 0; k < top; ++k) {
+    if (idx[tok * top + k] >= E) continue;
+    for (int i = threadIdx.x; i < ff; i += blockDim.x) sm[k * ff + i] = ldf(a + (tok * top + k) * ff + i);
+  }
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int per = (n + gridDim.y - 1) / gridDim.y;
   const int c0 = blockIdx.y * per, c1 = min(n, c0 + per);
-  for (int c = c0 + warp; c < c1; c += nw) {
-    float acc = 0.f;
+  for (int c = c0 + warp; c < c1; c += 2 * nw) {  // two rows per turn; the lanes' shares of all experts are added up once
+    const int c2 = c + nw < c1 ? c + nw : c;
+    float acc = 0.f, acc2 = 0.f;
     for (int k = 0; k < top; ++k) {
       const int e = idx[tok * top + k];
       if (e >= E) continue;
-      acc += (win ? 1.f : wts[tok * top + k]) * warp_dot<T>(wd + ((long)e * n + c) * ff, sm + k * ff, ff, lane);
+      const float wk = win ? 1.f : wts[tok * top + k];
+      const float2 d = lane_dot2<T>(wd + ((long)e * n + c) * ff, wd + ((long)e * n + c2) * ff, sm + k * ff, ff, lane);
+      acc += wk * d.x;
+      acc2 += wk * d.y;
     }
-    if (lane == 0) out[tok * n + c] = acc;
+    acc = warp_sum(acc);
+    acc2 = warp_sum(acc2);
+    if (lane == 0) {
+      out[tok * n + c] = acc;
+      if (c2 != c) out[tok * n + c2] = acc2;
+    }
   }
 }
 
