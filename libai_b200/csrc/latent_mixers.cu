@@ -408,7 +408,7 @@ latent_prompt_mma_kernel(const bf16* __restrict__ q, long ldq, const bf16* __res
 
 // ------------------------------------------------------------------------------------------------------------------
 // Absorbed form, step 1: qa[t, h, :C] = sum_d q[t, h, d] W_uk[h*D + d, :], qa[t, h, C:C+R] = the rotated query part (fp32).
-// Block (head, 128 channels, BT rows): four groups of 64 threads share the D rows of the head's matrix, two channels per thread.
+// Block (head, 64 channels, BT rows): the eight warps share the D rows of the head's matrix, two channels per lane.
 // ------------------------------------------------------------------------------------------------------------------
 template <typename T, int BT>
 __global__ void __launch_bounds__(256)
@@ -416,8 +416,8 @@ latent_absorb_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ wu
                      long rows, int H, int D, int R, int C) {
   extern __shared__ float sm[];
   float* qs = sm;                                // [BT][D]
-  float* red = sm + BT * D;                      // [3][BT][128]
-  const int h = blockIdx.x, c0 = blockIdx.y * 128, tid = threadIdx.x, grp = tid >> 6, c = c0 + (tid & 63) * 2;
+  float* red = sm + BT * D;                      // [7][BT][64]
+  const int h = blockIdx.x, c0 = blockIdx.y * 64, tid = threadIdx.x, grp = tid >> 5, lane = tid & 31, c = c0 + lane * 2;
   const long t0 = (long)blockIdx.z * BT;
   const int nt = (int)min((long)BT, rows - t0);
   const int CA = C + R;
@@ -437,13 +437,13 @@ latent_absorb_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ wu
     }
   }
   __syncthreads();
-  const int per = (D + 3) / 4, d0 = grp * per, d1 = min(D, d0 + per);
+  const int per = (D + 7) / 8, d0 = grp * per, d1 = min(D, d0 + per);
   float a0[BT], a1[BT];
 #pragma unroll
   for (int r = 0; r < BT; ++r) { a0[r] = a1[r] = 0.f; }
   if (c < C) {
     const bool two = c + 1 < C, wide = two && sizeof(T) == 2 && (C & 1) == 0 && (reinterpret_cast<uintptr_t>(wuk) & 3) == 0;
-#pragma unroll 4
+#pragma unroll 8
     for (int d = d0; d < d1; ++d) {
       const T* wr = wuk + ((long)h * D + d) * C + c;
       float w0, w1;
@@ -459,14 +459,14 @@ latent_absorb_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ wu
   }
   if (grp) {
 #pragma unroll
-    for (int r = 0; r < BT; ++r) { float* dst = red + ((grp - 1) * BT + r) * 128 + (tid & 63) * 2; dst[0] = a0[r]; dst[1] = a1[r]; }
+    for (int r = 0; r < BT; ++r) { float* dst = red + ((grp - 1) * BT + r) * 64 + lane * 2; dst[0] = a0[r]; dst[1] = a1[r]; }
   }
   __syncthreads();
   if (grp == 0 && c < C) {
 #pragma unroll
     for (int r = 0; r < BT; ++r) {
       if (r < nt) {
-        for (int g = 0; g < 3; ++g) { const float* src = red + (g * BT + r) * 128 + (tid & 63) * 2; a0[r] += src[0]; a1[r] += src[1]; }
+        for (int g = 0; g < 7; ++g) { const float* src = red + (g * BT + r) * 64 + lane * 2; a0[r] += src[0]; a1[r] += src[1]; }
         float* dst = qa + ((t0 + r) * H + h) * CA + c;
         dst[0] = a0[r];
         if (c + 1 < C) dst[1] = a1[r];
@@ -722,24 +722,34 @@ latent_absorbed_mma_kernel(const float* __restrict__ qa, const bf16* __restrict_
 
 // ------------------------------------------------------------------------------------------------------------------
 // Absorbed form, step 3: merge the parts of BT rows of one head (the sink joins the denominator) and apply the value
-// up-projection, y[t, h*V + v] = sum_c W_uv[h*V + v, c] lat[t, c]; a warp per value channel.
+// up-projection, y[t, h*V + v] = sum_c W_uv[h*V + v, c] lat[t, c]; a warp takes four value channels per turn.  The parts that hold
+// keys are the first ones of a row.
 // ------------------------------------------------------------------------------------------------------------------
 template <typename T, int BT>
 __global__ void __launch_bounds__(256)
 latent_value_kernel(const float* __restrict__ part, int nparts, const float* __restrict__ sink, const T* __restrict__ wuv, T* __restrict__ y,
                     long ldy, long rows, int H, int V, int C) {
-  extern __shared__ float sm[];
-  float* lat = sm;                               // [BT][C]
-  float* wt = sm + BT * C;                       // [BT][nparts] weight of every part
+  extern __shared__ __align__(16) float sm[];
+  __shared__ int used_s[BT];
+  const int CP = (C + 3) & ~3;
+  float* lat = sm;                               // [BT][CP]
+  float* wt = sm + BT * CP;                      // [BT][nparts] weight of every part
   const int h = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const long t0 = (long)blockIdx.y * BT;
   const int nt = (int)min((long)BT, rows - t0);
   const long step = C + 2;
-  if (warp < BT && warp < nt) {
+  if (warp < nt) {
     const float* base = part + (((t0 + warp) * H + h) * nparts) * step;
     float M = sink ? sink[h] : -INFINITY;
-    for (int s = lane; s < nparts; s += 32) M = fmaxf(M, base[s * step]);
+    int used = 0;
+    for (int s = lane; s < nparts; s += 32) {
+      const float m = base[s * step];
+      M = fmaxf(M, m);
+      if (m != -INFINITY) used = s + 1;
+    }
     M = warp_max(M);
+#pragma unroll
+    for (int mk = 16; mk > 0; mk >>= 1) used = max(used, __shfl_xor_sync(0xffffffffu, used, mk));
     float L = 0.f;
     for (int s = lane; s < nparts; s += 32) {
       const float w = expf(base[s * step] - M);  // an empty part has maximum -inf: weight 0
@@ -748,49 +758,65 @@ latent_value_kernel(const float* __restrict__ part, int nparts, const float* __r
     }
     L = warp_sum(L) + (sink ? expf(sink[h] - M) : 0.f);
     for (int s = lane; s < nparts; s += 32) wt[warp * nparts + s] /= L;
+    if (lane == 0) used_s[warp] = used;
   }
   __syncthreads();
-  for (int i = tid; i < BT * C; i += 256) {
-    const int r = i / C, c = i - r * C;
+  for (int i = tid; i < BT * CP; i += 256) {
+    const int r = i / CP, c = i - r * CP;
     float a = 0.f;
-    if (r < nt) {
+    if (r < nt && c < C) {
       const float* base = part + (((t0 + r) * H + h) * nparts) * step + 2 + c;
-      for (int s = 0; s < nparts; ++s) {
-        const float w = wt[r * nparts + s];
-        if (w != 0.f) a += w * base[s * step];
-      }
+      const int used = used_s[r];
+#pragma unroll 8
+      for (int s = 0; s < used; ++s) a += wt[r * nparts + s] * base[s * step];
     }
     lat[i] = a;
   }
   __syncthreads();
   constexpr int PV = sizeof(T) == 2 ? 8 : 4;
   const bool vec = C % PV == 0 && (reinterpret_cast<uintptr_t>(wuv) & 15) == 0;
-  for (int v = blockIdx.z * 8 + warp; v < V; v += 8 * gridDim.z) {
-    const T* wr = wuv + ((long)h * V + v) * C;
-    float acc[BT];
+  for (int v0 = (blockIdx.z * 8 + warp) * 4; v0 < V; v0 += 32 * gridDim.z) {
+    const T* wr[4];
 #pragma unroll
-    for (int r = 0; r < BT; ++r) acc[r] = 0.f;
+    for (int k = 0; k < 4; ++k) wr[k] = wuv + ((long)h * V + min(v0 + k, V - 1)) * C;
+    float acc[4][BT];
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+#pragma unroll
+      for (int r = 0; r < BT; ++r) acc[k][r] = 0.f;
     if (vec) {
 #pragma unroll 2
       for (int c = lane * PV; c < C; c += 32 * PV) {
-        float w[PV];
-        Pack<T, PV>::ld(wr + c, w);
+        float w[4][PV];
 #pragma unroll
-        for (int r = 0; r < BT; ++r)
+        for (int k = 0; k < 4; ++k) Pack<T, PV>::ld(wr[k] + c, w[k]);
 #pragma unroll
-          for (int e = 0; e < PV; ++e) acc[r] += w[e] * lat[r * C + c + e];
+        for (int r = 0; r < BT; ++r) {
+#pragma unroll
+          for (int e = 0; e < PV; e += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(lat + r * CP + c + e);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) acc[k][r] += w[k][e] * x.x + w[k][e + 1] * x.y + w[k][e + 2] * x.z + w[k][e + 3] * x.w;
+          }
+        }
       }
     } else {
       for (int c = lane; c < C; c += 32) {
-        const float w = ldf(wr + c);
 #pragma unroll
-        for (int r = 0; r < BT; ++r) acc[r] += w * lat[r * C + c];
+        for (int k = 0; k < 4; ++k) {
+          const float w = ldf(wr[k] + c);
+#pragma unroll
+          for (int r = 0; r < BT; ++r) acc[k][r] += w * lat[r * CP + c];
+        }
       }
     }
 #pragma unroll
-    for (int r = 0; r < BT; ++r) {
-      const float a = warp_sum(acc[r]);
-      if (lane == 0 && r < nt) stf(y + (t0 + r) * ldy + (long)h * V + v, a);
+    for (int k = 0; k < 4; ++k) {
+#pragma unroll
+      for (int r = 0; r < BT; ++r) {
+        const float a = warp_sum(acc[k][r]);
+        if (lane == 0 && r < nt && v0 + k < V) stf(y + (t0 + r) * ldy + (long)h * V + v0 + k, a);
+      }
     }
   }
 }
@@ -881,9 +907,9 @@ int lbl_latent_absorb(const void* q, long ldq, const void* wuk, const float* cs,
                       cudaStream_t s) {
   if (rows == 0) return 0;
   const int bt = rows >= 8 ? 8 : (rows >= 3 ? 4 : (rows == 2 ? 2 : 1));
-  const size_t smem = ((size_t)bt * D + 3 * (size_t)bt * 128) * sizeof(float);
+  const size_t smem = ((size_t)bt * D + 7 * (size_t)bt * 64) * sizeof(float);
   if (smem > 200 * 1024 || rows / bt > 60000) return -1;
-  const dim3 grid((unsigned)H, (unsigned)((C + 127) / 128), (unsigned)((rows + bt - 1) / bt));
+  const dim3 grid((unsigned)H, (unsigned)((C + 63) / 64), (unsigned)((rows + bt - 1) / bt));
 #define AB(TT, B_) { allow_smem(latent_absorb_kernel<TT, B_>, smem); \
     latent_absorb_kernel<TT, B_><<<grid, 256, smem, s>>>((const TT*)q, ldq, (const TT*)wuk, (const float2*)cs, qa, rows, H, D, R, C); }
 #define ABT(TT) { if (bt == 8) AB(TT, 8) else if (bt == 4) AB(TT, 4) else if (bt == 2) AB(TT, 2) else AB(TT, 1) }
@@ -931,7 +957,7 @@ int lbl_latent_value(const float* part, int nparts, const float* sink, const voi
                      int dtype, cudaStream_t s) {
   if (rows == 0) return 0;
   const int bt = rows * H >= 2048 ? 4 : 1;
-  const size_t smem = ((size_t)bt * C + (size_t)bt * nparts) * sizeof(float);
+  const size_t smem = ((size_t)bt * (C + 4) + (size_t)bt * nparts) * sizeof(float);
   const long groups = (rows + bt - 1) / bt;
   if (smem > 200 * 1024 || groups > 60000) return -1;
   int vz = (int)(148 / (groups * H)); if (vz > (V + 31) / 32) vz = (V + 31) / 32; if (vz < 1) vz = 1;

@@ -164,7 +164,7 @@ def latent_absorbed(q, wuk, wuv, cs, pool, table, rb, y, H: int, D: int, R: int,
         mma = mma and q.dtype == torch.bfloat16 and pool.data_ptr() % 16 == 0 and ext.latent_absorbed_mma_ok(C, R, pool.shape[2])
         if parts is None:
             groups = q.shape[0] * -(-H // (16 if mma else 8))
-            parts = max(1, min(64, -(-148 // groups) if mma else -(-592 // groups)))
+            parts = max(1, min(64, 148 // groups if mma else -(-592 // groups)))     # mma: one wave of one block per SM
         count_launch(3)
         ext.latent_absorbed(q, wuk, wuv, cs, sink, pool, table, rb.tok_seq, rb.seq_off, rb.slots, rb.past, y, H, D, R, V, C, float(scale), parts, mma)
         return y
