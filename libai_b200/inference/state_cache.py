@@ -10,7 +10,7 @@ A model registers one entry per layer run (a layer that is run several times in 
 * ``"recurrent"`` — the matrix state of a delta-rule or linear-attention layer, ``[slots, H, D, V]`` in fp32, and the last
   ``taps - 1`` inputs of its short convolutions, ``[slots, taps - 1, C]`` (empty for a layer without convolutions);
 * ``"token"`` — the last token of the sequence, ``[slots]`` int32 (an embedding that looks at the previous token);
-* ``"paged"`` — the key/value rows of an attention layer that sees the whole past: a pool ``[pages, page_size, C]`` in the compute
+* ``"paged"`` — the key/value rows (or latent rows) of an attention layer that sees the whole past: a pool ``[pages, page_size, C]`` in the compute
   dtype, shared by all sequences, and the last ``taps - 1`` inputs of the layer's short convolutions,
   ``[slots, taps - 1, conv_channels]``.  Position ``p`` of a sequence lives in row ``p % page_size`` of page
   ``page_table[slot, p // page_size]``; all paged entries share one page table (a page id names the same page of every pool).

@@ -1,6 +1,6 @@
 """In-tree build of the native extensions: ``libai_b200/_C.so`` (GEMM, attention, norms, optimizer, collectives) and
 ``libai_b200/_C_seq.so`` (ragged-batch sequence mixers with per-sequence state), ``libai_b200/_C_kv.so`` (ring and paged key/value
-caches, masked grouped-query attention, attention with mixed heads, Dynamic-Tanh and post-norm residuals, mixture of experts) and ``libai_b200/_C_lin.so`` (bigram embedding,
+caches, masked grouped-query attention, attention with mixed heads, attention on paged latents, Dynamic-Tanh and post-norm residuals, mixture of experts) and ``libai_b200/_C_lin.so`` (bigram embedding,
 hyper-connection streams, decayed linear-attention recurrences).
 
     python -m libai_b200.ops.build [--force] [--verbose] [--only _C|_C_seq|_C_kv|_C_lin]
