@@ -27,16 +27,21 @@ int lbk_masked_attention(const void* q, long ldq, const void* kbase, const void*
                          int L, int nfirst, const int* ext_off, const int* nsink, const int* cstart, const int* slots,
                          const void* gate, long ldg, const int* tok_seq, const int* seq_off, const int* past, void* y, long ldy,
                          long tokens, int H, int G, int D, int V, int window, int chunk, int keep, float scale, float softcap,
-                         int sink, int gate_wide, float out_scale, int dtype, cudaStream_t s);
+                         int sink, int gate_wide, float out_scale, float temp_coef, float temp_every, const void* pool, const int* table,
+                         int max_pages, int page, int dtype, cudaStream_t s);
 int lbk_masked_attention_mma(const void* q, long ldq, const void* kbase, const void* vbase, long ldkv, const int* ext_off,
                              const int* nsink, const int* cstart, const void* gate, long ldg, const int* qt_seq, const int* qt_start,
                              int n_qtiles, const int* seq_off, const int* past, void* y, long ldy, int H, int G, int D, int V,
                              int window, int chunk, int keep, float scale, float softcap, int sink, int gate_wide, float out_scale,
-                             cudaStream_t s);
+                             float temp_coef, float temp_every, cudaStream_t s);
 int lbk_ring_decode(const void* q, long ldq, const void* ring, const void* first, int L, int nfirst, const int* slots, const int* past,
                     const void* gate, long ldg, void* y, long ldy, float* part, int B, int H, int G, int D, int V, int window,
-                    int chunk, int keep, float scale, int splits, float softcap, int sink, int gate_wide, float out_scale, int dtype,
-                    cudaStream_t s);
+                    int chunk, int keep, float scale, int splits, float softcap, int sink, int gate_wide, float out_scale, float temp_coef,
+                    float temp_every, const int* table, int max_pages, int page, int dtype, cudaStream_t s);
+int lbk_heads_prepare(void* q, long ldq, void* k, long ldk, const void* v, long ldv, const void* qn, const void* kn, const float* freq,
+                      int half, int pairs, float eps, void* base, int L, const int* table, int max_pages, int page, const int* tok_seq,
+                      const int* seq_off, const int* slots, const int* past, long tokens, int H, int G, int D, int V, int dtype,
+                      cudaStream_t s);
 int lbk_moe_topk(const float* z, long ldz, const float* bias, const float* corr, int mode, int E, int real, int top, float rscale, int* idx,
                  float* wts, int* counts, float* keep, long tokens, cudaStream_t s);
 int lbk_moe_pairs(const void* h, long ldh, const void* wgu, const void* wd, const int* idx, const float* wts, void* a, float* out,
@@ -47,6 +52,9 @@ int lbp_postnorm_residual(const float* xin, float* xout, const void* y1, long ld
                           const int* pos, const float* cw, int top, float alpha, const float* gate, long ldgate, const float* keep,
                           int outer, float out_scale, const void* w, float eps, void* h, long ldh, long rows, int n, int dtype,
                           cudaStream_t s);
+int lbp_sandwich_residual(float* x, const float* y, long ldy, const float* y2, long ldy2, const void* bw1, const void* bw2, float bscale,
+                          const void* pw, float mult, const void* add, const void* nw, float eps, void* h, long ldh, long rows, int n,
+                          int dtype, cudaStream_t s);
 int lbp_conv_qkv_prepare(const void* qin, const void* kin, const void* vin, long ld, const void* wq, const void* wk, const void* wv,
                          int taps, void* tail, const void* qn, const void* kn, const float* freq, int half, float eps, void* qout,
                          long ldqo, void* pool, const int* table, int max_pages, int page_size, const int* tok_seq,
@@ -201,7 +209,8 @@ void kv_gather(const Tensor& ring, const Tensor& first, const Tensor& knew, cons
 void masked_attention(const Tensor& q, const Tensor& kmat, const Tensor& vmat, const Tensor& ext_off, const Tensor& nsink,
                       const Tensor& cstart, const OptT& gate, const Tensor& tok_seq, const Tensor& seq_off, const Tensor& past,
                       const OptT& qt_seq, const OptT& qt_start, Tensor y, int64_t H, int64_t G, int64_t D, int64_t V, int64_t window,
-                      int64_t chunk, int64_t keep, double scale, double softcap, bool sink, bool gate_wide, double out_scale) {
+                      int64_t chunk, int64_t keep, double scale, double softcap, bool sink, bool gate_wide, double out_scale,
+                      double temp_coef, double temp_every) {
   rows2d(q, "masked_attention q"); rows2d(kmat, "masked_attention k"); rows2d(vmat, "masked_attention v"); rows2d(y, "masked_attention y");
   const int dtype = code(q);
   TORCH_CHECK(q.size(1) == H * D && kmat.size(1) == G * D && vmat.size(1) == G * V && y.size(1) == H * V && y.size(0) == q.size(0) &&
@@ -214,21 +223,24 @@ void masked_attention(const Tensor& q, const Tensor& kmat, const Tensor& vmat, c
     check(lbk_masked_attention_mma(q.data_ptr(), q.stride(0), kmat.data_ptr(), vmat.data_ptr(), kmat.stride(0), meta(ext_off), meta(nsink),
                                    meta(cstart), ptr_opt(gate), ldg, meta(*qt_seq), meta(*qt_start), (int)qt_seq->numel(), meta(seq_off),
                                    meta(past), y.data_ptr(), y.stride(0), (int)H, (int)G, (int)D, (int)V, (int)window, (int)chunk, (int)keep,
-                                   (float)scale, (float)softcap, (int)sink, (int)gate_wide, (float)out_scale, cur_stream()),
+                                   (float)scale, (float)softcap, (int)sink, (int)gate_wide, (float)out_scale, (float)temp_coef, (float)temp_every,
+                                   cur_stream()),
           "masked_attention (tensor cores)");
     return;
   }
   check(lbk_masked_attention(q.data_ptr(), q.stride(0), kmat.data_ptr(), vmat.data_ptr(), kmat.stride(0), nullptr, nullptr, 0, 0,
                              meta(ext_off), meta(nsink), meta(cstart), nullptr, ptr_opt(gate), ldg, meta(tok_seq), meta(seq_off), meta(past),
                              y.data_ptr(), y.stride(0), q.size(0), (int)H, (int)G, (int)D, (int)V, (int)window, (int)chunk, (int)keep,
-                             (float)scale, (float)softcap, (int)sink, (int)gate_wide, (float)out_scale, dtype, cur_stream()), "masked_attention");
+                             (float)scale, (float)softcap, (int)sink, (int)gate_wide, (float)out_scale, (float)temp_coef, (float)temp_every, nullptr,
+                             nullptr, 0, 0, dtype, cur_stream()), "masked_attention");
 }
 
 // single-token steps: keys / values straight from the ring and the kept-first rows.  splits == 0: one warp per (token, head);
 // splits > 0: the grouped kernel, the keys of a (sequence, key head) cut into `splits` parts and merged.
 void ring_attention(const Tensor& q, const Tensor& ring, const Tensor& first, const OptT& gate, const Tensor& tok_seq, const Tensor& seq_off,
                     const Tensor& slots, const Tensor& past, Tensor y, int64_t H, int64_t G, int64_t D, int64_t V, int64_t window,
-                    int64_t chunk, int64_t keep, double scale, int64_t splits, double softcap, bool sink, bool gate_wide, double out_scale) {
+                    int64_t chunk, int64_t keep, double scale, int64_t splits, double softcap, bool sink, bool gate_wide, double out_scale,
+                    double temp_coef, double temp_every) {
   rows2d(q, "ring_attention q"); rows2d(y, "ring_attention y");
   const int dtype = code(q);
   ring_shapes(ring, first, G * (D + V));
@@ -242,14 +254,68 @@ void ring_attention(const Tensor& q, const Tensor& ring, const Tensor& first, co
     check(lbk_ring_decode(q.data_ptr(), q.stride(0), ring.data_ptr(), first.data_ptr(), (int)ring.size(1), (int)first.size(1), meta(slots),
                           meta(past), ptr_opt(gate), ldg, y.data_ptr(), y.stride(0), part.data_ptr<float>(), (int)q.size(0), (int)H, (int)G,
                           (int)D, (int)V, (int)window, (int)chunk, (int)keep, (float)scale, (int)splits, (float)softcap, (int)sink, (int)gate_wide,
-                          (float)out_scale, dtype, cur_stream()), "ring_decode");
+                          (float)out_scale, (float)temp_coef, (float)temp_every, nullptr, 0, 0, dtype, cur_stream()), "ring_decode");
     return;
   }
   check(lbk_masked_attention(q.data_ptr(), q.stride(0), nullptr, nullptr, 0, ring.data_ptr(), first.data_ptr(), (int)ring.size(1),
                              (int)first.size(1), nullptr, nullptr, nullptr, meta(slots), ptr_opt(gate), ldg, meta(tok_seq), meta(seq_off),
                              meta(past), y.data_ptr(), y.stride(0), q.size(0), (int)H, (int)G, (int)D, (int)V, (int)window, (int)chunk,
-                             (int)keep, (float)scale, (float)softcap, (int)sink, (int)gate_wide, (float)out_scale, dtype, cur_stream()),
-        "ring_attention");
+                             (int)keep, (float)scale, (float)softcap, (int)sink, (int)gate_wide, (float)out_scale, (float)temp_coef,
+                             (float)temp_every, nullptr, nullptr, 0, 0, dtype, cur_stream()), "ring_attention");
+}
+
+// single-token steps over a paged cache: pool [pages, page_size, G*D + G*V], table int32 [slots, max_pages]; the whole past is visible
+void page_attention(const Tensor& q, const Tensor& pool, const Tensor& table, const OptT& gate, const Tensor& tok_seq, const Tensor& seq_off,
+                    const Tensor& slots, const Tensor& past, Tensor y, int64_t H, int64_t G, int64_t D, int64_t V, double scale, int64_t splits,
+                    double softcap, bool sink, bool gate_wide, double out_scale, double temp_coef, double temp_every) {
+  rows2d(q, "page_attention q"); rows2d(y, "page_attention y");
+  const int dtype = code(q);
+  TORCH_CHECK(pool.is_cuda() && pool.dim() == 3 && pool.is_contiguous() && pool.size(2) == G * (D + V) && code(pool) == dtype && table.dim() == 2,
+              "page_attention: pool [pages, page_size, G*D + G*V], table [slots, max_pages]");
+  TORCH_CHECK(q.size(1) == H * D && y.size(1) == H * V && y.size(0) == q.size(0) && code(y) == dtype && q.size(0) == slots.numel(),
+              "page_attention: shapes (one token per sequence)");
+  long ldg = 0;
+  if (has(gate)) { rows2d(*gate, "page_attention gate"); TORCH_CHECK(gate->size(1) == (gate_wide ? H * V : H) && code(*gate) == dtype, "page_attention: gate [tokens, H] (or [tokens, H V])"); ldg = gate->stride(0); }
+  c10::cuda::CUDAGuard guard(q.device());
+  if (splits > 0) {
+    Tensor part = at::empty({q.size(0) * H * splits * (V + 2)}, q.options().dtype(at::kFloat));
+    check(lbk_ring_decode(q.data_ptr(), q.stride(0), pool.data_ptr(), nullptr, 1, 0, meta(slots), meta(past), ptr_opt(gate), ldg, y.data_ptr(),
+                          y.stride(0), part.data_ptr<float>(), (int)q.size(0), (int)H, (int)G, (int)D, (int)V, 0, 0, 0, (float)scale, (int)splits,
+                          (float)softcap, (int)sink, (int)gate_wide, (float)out_scale, (float)temp_coef, (float)temp_every, meta(table),
+                          (int)table.size(1), (int)pool.size(1), dtype, cur_stream()), "page_attention");
+    return;
+  }
+  check(lbk_masked_attention(q.data_ptr(), q.stride(0), nullptr, nullptr, 0, nullptr, nullptr, 0, 0, nullptr, nullptr, nullptr, meta(slots),
+                             ptr_opt(gate), ldg, meta(tok_seq), meta(seq_off), meta(past), y.data_ptr(), y.stride(0), q.size(0), (int)H, (int)G,
+                             (int)D, (int)V, 0, 0, 0, (float)scale, (float)softcap, (int)sink, (int)gate_wide, (float)out_scale, (float)temp_coef,
+                             (float)temp_every, pool.data_ptr(), meta(table), (int)table.size(1), (int)pool.size(1), dtype, cur_stream()),
+        "page_attention");
+}
+
+// per-head norm and rotation of q and k in place; keys and values to `cache`: a ring [slots, L, C] (no table) or pages (table given)
+void heads_prepare(Tensor q, Tensor k, const Tensor& v, const OptT& qn, const OptT& kn, const Tensor& freq, bool pairs, double eps,
+                   const OptT& cache, const OptT& table, const Tensor& tok_seq, const Tensor& seq_off, const Tensor& slots, const Tensor& past,
+                   int64_t H, int64_t G, int64_t D, int64_t V) {
+  rows2d(q, "heads_prepare q"); rows2d(k, "heads_prepare k"); rows2d(v, "heads_prepare v");
+  const int dtype = code(q);
+  const int64_t tokens = q.size(0);
+  TORCH_CHECK(q.size(1) == H * D && k.size(1) == G * D && v.size(1) == G * V && k.size(0) == tokens && v.size(0) == tokens && code(k) == dtype &&
+              code(v) == dtype, "heads_prepare: q [tokens, H*D], k [tokens, G*D], v [tokens, G*V]");
+  TORCH_CHECK(has(qn) == has(kn), "heads_prepare: both norm weights or none");
+  if (has(qn)) { vec(*qn, D, dtype, "heads_prepare q norm"); vec(*kn, D, dtype, "heads_prepare k norm"); }
+  TORCH_CHECK(freq.is_cuda() && freq.scalar_type() == at::kFloat && freq.is_contiguous() && 2 * freq.numel() <= D, "heads_prepare: freq fp32 [rotated channels / 2]");
+  void* base = nullptr; const int* tp = nullptr; int L = 0, max_pages = 0, page = 0;
+  if (has(cache)) {
+    TORCH_CHECK(cache->is_cuda() && cache->is_contiguous() && cache->dim() == 3 && cache->size(2) == G * (D + V) && code(*cache) == dtype,
+                "heads_prepare: cache rows [*, *, G*D + G*V]");
+    base = cache->data_ptr();
+    if (has(table)) { TORCH_CHECK(table->dim() == 2, "heads_prepare: table [slots, max_pages]"); tp = meta(*table); max_pages = (int)table->size(1); page = (int)cache->size(1); }
+    else L = (int)cache->size(1);
+  }
+  c10::cuda::CUDAGuard guard(q.device());
+  check(lbk_heads_prepare(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), ptr_opt(qn), ptr_opt(kn),
+                          freq.data_ptr<float>(), (int)freq.numel(), pairs ? 1 : 0, (float)eps, base, L, tp, max_pages, page, meta(tok_seq),
+                          meta(seq_off), meta(slots), meta(past), tokens, (int)H, (int)G, (int)D, (int)V, dtype, cur_stream()), "heads_prepare");
 }
 
 // E: how many leading columns of z are choices (-1: all); the first `real` of them are experts, the rest identity experts
@@ -370,6 +436,43 @@ void postnorm_residual(const Tensor& x, const OptT& xout, const OptT& y1, const 
                               outer ? 1 : 0, (float)out_scale, w.data_ptr(), (float)eps, hp, ldh, rows, (int)n, dtype, cur_stream()), "postnorm_residual");
 }
 
+// x fp32 [rows, n] in place: x += mult * rmsnorm(v) (1 + post) with v = y, or — y2 given — bscale * (rmsnorm(y) bw1 + rmsnorm(y2) bw2);
+// x += add (one row for all); h = rmsnorm(x) (1 + next).  Every step is optional
+void sandwich_residual(Tensor x, const OptT& y, const OptT& y2, const OptT& bw1, const OptT& bw2, double bscale, const OptT& post, double mult,
+                       const OptT& add, const OptT& next, double eps, const OptT& h) {
+  TORCH_CHECK(x.is_cuda() && x.dim() == 2 && x.is_contiguous() && x.scalar_type() == at::kFloat, "sandwich_residual: x fp32 [rows, width]");
+  const int64_t rows = x.size(0), n = x.size(1);
+  int dtype = -1;
+  auto weight = [&](const OptT& w, const char* name) -> const void* {
+    if (!has(w)) return nullptr;
+    if (dtype < 0) dtype = code(*w);
+    vec(*w, n, dtype, name);
+    return w->data_ptr();
+  };
+  const void *pw = weight(post, "sandwich_residual post"), *b1 = weight(bw1, "sandwich_residual bw1"), *b2 = weight(bw2, "sandwich_residual bw2"),
+             *ap = weight(add, "sandwich_residual add"), *nw = weight(next, "sandwich_residual next");
+  const float *yp = nullptr, *y2p = nullptr; long ldy = 0, ldy2 = 0;
+  auto rowsf = [&](const OptT& t, const char* name, long& ld) -> const float* {
+    if (!has(t)) return nullptr;
+    rows2d(*t, name);
+    TORCH_CHECK(t->scalar_type() == at::kFloat && t->size(0) == rows && t->size(1) == n, name, ": fp32 [rows, width] expected");
+    ld = t->stride(0);
+    return t->data_ptr<float>();
+  };
+  yp = rowsf(y, "sandwich_residual y", ldy); y2p = rowsf(y2, "sandwich_residual y2", ldy2);
+  TORCH_CHECK((!yp || pw) && (!y2p || (yp && b1 && b2)) && has(h) == (nw != nullptr), "sandwich_residual: outputs and their norm weights");
+  void* hp = nullptr; long ldh = 0;
+  if (has(h)) {
+    rows2d(*h, "sandwich_residual h");
+    TORCH_CHECK(h->size(0) == rows && h->size(1) == n && code(*h) == dtype, "sandwich_residual: h [rows, width] of the weights' dtype");
+    hp = h->data_ptr(); ldh = h->stride(0);
+  }
+  TORCH_CHECK(dtype >= 0, "sandwich_residual: nothing to do");
+  c10::cuda::CUDAGuard guard(x.device());
+  check(lbp_sandwich_residual(x.data_ptr<float>(), yp, ldy, y2p, ldy2, b1, b2, (float)bscale, pw, (float)mult, ap, nw, (float)eps, hp, ldh, rows, (int)n,
+                              dtype, cur_stream()), "sandwich_residual");
+}
+
 // q, k, v: column slices of one projection output (one row stride).  tail [slots, taps-1, H*D + G*D + G*V]; pool
 // [pages, page_size, G*D + G*V]; table int32 [slots, max_pages]
 void conv_qkv_prepare(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& wq, const Tensor& wk, const Tensor& wv, Tensor tail,
@@ -448,12 +551,15 @@ TORCH_LIBRARY(libai_b200_kv, m) {
   m.def("qk_prepare(Tensor(a!) q, Tensor(b!)? k, Tensor? qw, Tensor? kw, Tensor freq, float mscale, int H, int G, int D, float eps, bool full_norm, bool unit_norm, Tensor tok_seq, Tensor seq_off, Tensor past) -> ()", &qk_prepare);
   m.def("kv_write(Tensor(a!) ring, Tensor(b!) first, Tensor knew, Tensor vnew, Tensor tok_seq, Tensor seq_off, Tensor slots, Tensor past) -> ()", &kv_write);
   m.def("kv_gather(Tensor ring, Tensor first, Tensor knew, Tensor vnew, Tensor ext_seq, Tensor ext_off, Tensor nsink, Tensor cstart, Tensor seq_off, Tensor slots, Tensor past, Tensor(a!) ext) -> ()", &kv_gather);
-  m.def("masked_attention(Tensor q, Tensor kmat, Tensor vmat, Tensor ext_off, Tensor nsink, Tensor cstart, Tensor? gate, Tensor tok_seq, Tensor seq_off, Tensor past, Tensor? qt_seq, Tensor? qt_start, Tensor(a!) y, int H, int G, int D, int V, int window, int chunk, int keep, float scale, float softcap=0.0, bool sink=False, bool gate_wide=False, float out_scale=1.0) -> ()", &masked_attention);
-  m.def("ring_attention(Tensor q, Tensor ring, Tensor first, Tensor? gate, Tensor tok_seq, Tensor seq_off, Tensor slots, Tensor past, Tensor(a!) y, int H, int G, int D, int V, int window, int chunk, int keep, float scale, int splits, float softcap=0.0, bool sink=False, bool gate_wide=False, float out_scale=1.0) -> ()", &ring_attention);
+  m.def("masked_attention(Tensor q, Tensor kmat, Tensor vmat, Tensor ext_off, Tensor nsink, Tensor cstart, Tensor? gate, Tensor tok_seq, Tensor seq_off, Tensor past, Tensor? qt_seq, Tensor? qt_start, Tensor(a!) y, int H, int G, int D, int V, int window, int chunk, int keep, float scale, float softcap=0.0, bool sink=False, bool gate_wide=False, float out_scale=1.0, float temp_coef=0.0, float temp_every=0.0) -> ()", &masked_attention);
+  m.def("ring_attention(Tensor q, Tensor ring, Tensor first, Tensor? gate, Tensor tok_seq, Tensor seq_off, Tensor slots, Tensor past, Tensor(a!) y, int H, int G, int D, int V, int window, int chunk, int keep, float scale, int splits, float softcap=0.0, bool sink=False, bool gate_wide=False, float out_scale=1.0, float temp_coef=0.0, float temp_every=0.0) -> ()", &ring_attention);
+  m.def("page_attention(Tensor q, Tensor pool, Tensor table, Tensor? gate, Tensor tok_seq, Tensor seq_off, Tensor slots, Tensor past, Tensor(a!) y, int H, int G, int D, int V, float scale, int splits, float softcap=0.0, bool sink=False, bool gate_wide=False, float out_scale=1.0, float temp_coef=0.0, float temp_every=0.0) -> ()", &page_attention);
+  m.def("heads_prepare(Tensor(a!) q, Tensor(b!) k, Tensor v, Tensor? qn, Tensor? kn, Tensor freq, bool pairs, float eps, Tensor(c!)? cache, Tensor? table, Tensor tok_seq, Tensor seq_off, Tensor slots, Tensor past, int H, int G, int D, int V) -> ()", &heads_prepare);
   m.def("moe_topk(Tensor z, Tensor? bias, int mode, int top, float rscale, Tensor(a!) idx, Tensor(b!) wts, Tensor(c!)? counts, Tensor? corr=None, int E=-1, int real=-1, Tensor(d!)? keep=None) -> ()", &moe_topk);
   m.def("moe_pairs(Tensor h, Tensor wgu, Tensor wd, Tensor idx, Tensor wts, Tensor(a!) a, Tensor(b!) out, int act, float limit=0.0, bool weight_input=False, bool gated=True) -> ()", &moe_pairs);
   m.def("moe_sort(Tensor h, Tensor idx, Tensor counts, Tensor(a!) offsets, Tensor(b!) cursor, Tensor(c!) pos, Tensor(d!) xs, int align, Tensor(e!)? tile_group, Tensor? wts=None) -> ()", &moe_sort);
   m.def("postnorm_residual(Tensor x, Tensor(a!)? xout, Tensor? y1, Tensor? y2, Tensor? pos, Tensor? cw, float alpha, Tensor w, float eps, Tensor(b!)? h, Tensor? gate=None, Tensor? keep=None, bool outer=False, float out_scale=1.0) -> ()", &postnorm_residual);
+  m.def("sandwich_residual(Tensor(a!) x, Tensor? y, Tensor? y2, Tensor? bw1, Tensor? bw2, float bscale, Tensor? post, float mult, Tensor? add, Tensor? next, float eps, Tensor(b!)? h) -> ()", &sandwich_residual);
   m.def("conv_qkv_prepare(Tensor q, Tensor k, Tensor v, Tensor wq, Tensor wk, Tensor wv, Tensor(a!) tail, Tensor qn, Tensor kn, Tensor freq, float eps, Tensor(b!) qout, Tensor(c!) pool, Tensor table, Tensor tok_seq, Tensor seq_off, Tensor slots, Tensor past, int H, int G, int D, int V) -> ()", &conv_qkv_prepare);
   m.def("talk_attention_tiles(int qt_max, int H, int G, int D, int V) -> int[]", &talk_attention_tiles);
   m.def("talk_attention(Tensor q, Tensor pool, Tensor table, Tensor? talk, Tensor? sink, Tensor qt_seq, Tensor? qt_start, int QT, int KT, Tensor seq_off, Tensor slots, Tensor past, Tensor(a!) y, Tensor(b!)? part, int nparts, int H, int G, int D, int V, float scale, float out_scale) -> ()", &talk_attention);

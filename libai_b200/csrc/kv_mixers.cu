@@ -330,6 +330,118 @@ qk_prepare_kernel(T* __restrict__ q, long ldq, T* __restrict__ k, long ldk, cons
 }
 
 // ------------------------------------------------------------------------------------------------------------------
+// Head preparation with the cache write in the same pass: one warp per (token, group of `per` head units); the units of a token are
+// the H query heads, the G key heads and — when there is a cache to write — the G value heads.
+//   norm     : queries / keys divided by the root mean square of their head, times qn / kn [D] shared by the heads (optional)
+//   rotation : channel pairs (2i, 2i + 1) — `pairs` — or (i, i + half), i < half, turned by position * freq[i] (after the norm)
+// Queries and keys are rewritten in place (neither norm nor rotation: they are left alone and only copied).  Keys and values go to
+// the row [G*D | G*V] of their position: ring[slot][pos % L] (the last L new positions of a sequence) or the page row
+// table[slot][pos / page] * page + pos % page.  VEC: four consecutive channels per lane and access, `pairs` only.
+// ------------------------------------------------------------------------------------------------------------------
+struct CacheRows { void* base; const int* table; int L, max_pages, page, C, KC; };     // base: the ring (table null) or the pool
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(128)
+heads_prepare_kernel(T* __restrict__ q, long ldq, T* __restrict__ k, long ldk, const T* __restrict__ v, long ldv, const T* __restrict__ qn,
+                     const T* __restrict__ kn, const float* __restrict__ freq, int half, int pairs, float eps, CacheRows cr,
+                     const int* __restrict__ tok_seq, const int* __restrict__ seq_off, const int* __restrict__ slots,
+                     const int* __restrict__ past, long tokens, int H, int G, int D, int V, int unit0, int units, int per) {
+  constexpr int SL = QK_MAXD / 64;               // channel pairs per lane
+  const int lane = threadIdx.x & 31;
+  const long wid = (long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int groups = (units - unit0 + per - 1) / per;
+  const long tok = wid / groups;
+  if (tok >= tokens) return;
+  const int u0 = unit0 + (int)(wid - tok * groups) * per, u1 = min(units, u0 + per);
+  const int b = tok_seq[tok], t = (int)(tok - seq_off[b]), n = seq_off[b + 1] - seq_off[b], pos = past[b] + t;
+  T* row = nullptr;                               // this position's cache row
+  if (cr.base) {
+    const long slot = slots[b];
+    if (cr.table) row = (T*)cr.base + ((long)cr.table[slot * cr.max_pages + pos / cr.page] * cr.page + pos % cr.page) * cr.C;
+    else if (n - t <= cr.L) row = (T*)cr.base + (slot * cr.L + pos % cr.L) * cr.C;
+  }
+  float cs[SL], sn[SL];
+  int c0[SL], c1[SL];
+#pragma unroll
+  for (int j = 0; j < SL; ++j) {                  // pair slot -> its two channels
+    const int s = VEC ? (j >> 1) * 64 + lane * 2 + (j & 1) : lane + 32 * j;
+    const bool turned = s < half;
+    c0[j] = (turned && !pairs) ? s : 2 * s;
+    c1[j] = (turned && !pairs) ? s + half : 2 * s + 1;
+    cs[j] = 1.f; sn[j] = 0.f;
+    if (turned && u0 < H + G) sincosf((float)pos * freq[s], &sn[j], &cs[j]);
+  }
+  for (int u = u0; u < u1; ++u) {
+    const bool isq = u < H, isv = u >= H + G;
+    if (isv && !row) break;
+    const int hh = isq ? u : (isv ? u - H - G : u - H), W = isv ? V : D;
+    const T* src = isq ? q + tok * ldq + (long)hh * D : (isv ? v + tok * ldv + (long)hh * V : k + tok * ldk + (long)hh * D);
+    float a[SL], d[SL];
+    float ss = 0.f;
+    if (VEC) {
+#pragma unroll
+      for (int j = 0; j < SL; j += 2) {
+        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c0[j] < W) x = ld4<T>(src + c0[j]);
+        a[j] = x.x; d[j] = x.y; a[j + 1] = x.z; d[j + 1] = x.w;
+        ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < SL; ++j) {
+        // (a value head has no rotated channels: its pairs are consecutive)
+        const int e0 = isv ? 2 * (lane + 32 * j) : c0[j], e1 = isv ? e0 + 1 : c1[j];
+        a[j] = e0 < W ? ldf(src + e0) : 0.f; d[j] = e1 < W ? ldf(src + e1) : 0.f;
+        ss += a[j] * a[j] + d[j] * d[j];
+      }
+    }
+    if (!isv) {
+      const T* w = isq ? qn : kn;
+      if (w) {
+        const float r = 1.f / sqrtf(warp_sum(ss) / (float)D + eps);
+        if (VEC) {
+#pragma unroll
+          for (int j = 0; j < SL; j += 2) {
+            if (c0[j] < D) {
+              const float4 x = ld4<T>(w + c0[j]);
+              a[j] *= r * x.x; d[j] *= r * x.y; a[j + 1] *= r * x.z; d[j + 1] *= r * x.w;
+            }
+          }
+        } else {
+#pragma unroll
+          for (int j = 0; j < SL; ++j) { if (c0[j] < D) a[j] *= r * ldf(w + c0[j]); if (c1[j] < D) d[j] *= r * ldf(w + c1[j]); }
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < SL; ++j) {              // (unturned pairs: cos 1, sin 0)
+        const float x = a[j] * cs[j] - d[j] * sn[j], y = d[j] * cs[j] + a[j] * sn[j];
+        a[j] = x; d[j] = y;
+      }
+    }
+    T* dst = isv ? nullptr : (isq ? q + tok * ldq + (long)hh * D : k + tok * ldk + (long)hh * D);
+    T* keep = (isq || !row) ? nullptr : (isv ? row + cr.KC + hh * V : row + hh * D);
+    const bool rewrite = dst && unit0 == 0;
+    if (VEC) {
+#pragma unroll
+      for (int j = 0; j < SL; j += 2) {
+        if (c0[j] < W) {
+          const float4 x = make_float4(a[j], d[j], a[j + 1], d[j + 1]);
+          if (rewrite) st4<T>(dst + c0[j], x);
+          if (keep) st4<T>(keep + c0[j], x);
+        }
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < SL; ++j) {
+        const int e0 = isv ? 2 * (lane + 32 * j) : c0[j], e1 = isv ? e0 + 1 : c1[j];
+        if (e0 < W) { if (rewrite) stf(dst + e0, a[j]); if (keep) stf(keep + e0, a[j]); }
+        if (e1 < W) { if (rewrite) stf(dst + e1, d[j]); if (keep) stf(keep + e1, d[j]); }
+      }
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------------------
 // Cache rows.  kv_write: the step's key rows (G*D) and value rows (G*V) go to ring[slot][pos % L] (only the last L of a
 // sequence's new tokens) and, for pos < nfirst, to first[slot][pos].  kv_gather: builds the ext matrix of a prompt step.
 // ------------------------------------------------------------------------------------------------------------------
@@ -387,20 +499,29 @@ __global__ void kv_gather_kernel(const T* __restrict__ ring, const T* __restrict
 // Options of every attention kernel of this file (AttnExtra): `softcap` > 0 passes the scaled scores through
 // cap * tanh(score / cap); `sink` adds one entry of score 0 without a value to the softmax (its denominator grows by
 // exp(0)); `gate_wide` reads one gate logit per output channel (gate[tok, h*V + c]) instead of one per head; the result
-// is multiplied by `out_scale`.
+// is multiplied by `out_scale`; `temp_every` > 0 multiplies the query at position p by
+// 1 + temp_coef * ln(floor((p + 1) / temp_every) + 1).
 // ------------------------------------------------------------------------------------------------------------------
-struct AttnExtra { float softcap, out_scale; int sink, gate_wide; };
+struct AttnExtra { float softcap, out_scale; int sink, gate_wide; float temp_coef, temp_every; };
+__device__ __forceinline__ float query_temperature(int pos, float coef, float every) {
+  return every > 0.f ? 1.f + coef * logf(floorf((float)(pos + 1) / every) + 1.f) : 1.f;
+}
 constexpr int ATT_MAXV = 8;    // value channels per lane: V <= 256
 
 struct KvSource {
   const void* kbase; const void* vbase; long ldkv;            // ext mode
   const void* ring; const void* first; int L, nfirst, C, KC;  // ring mode
+  const void* pool; const int* table; int max_pages, page;    // page mode (table given)
   const int* ext_off; const int* nsink; const int* cstart; const int* slots;
 };
 
 template <typename T>
 __device__ __forceinline__ void kv_row(const KvSource& s, int b, int pos, int g, int D, int V, const T*& kp, const T*& vp) {
-  if (s.ring) {
+  if (s.table) {
+    const long slot = s.slots[b];
+    const T* base = (const T*)s.pool + ((long)s.table[slot * s.max_pages + pos / s.page] * s.page + pos % s.page) * s.C;
+    kp = base + g * D; vp = base + s.KC + g * V;
+  } else if (s.ring) {
     const long slot = s.slots[b];
     const T* base = pos < s.nfirst ? (const T*)s.first + (slot * s.nfirst + pos) * s.C : (const T*)s.ring + (slot * s.L + pos % s.L) * s.C;
     kp = base + g * D; vp = base + s.KC + g * V;
@@ -429,6 +550,7 @@ __global__ void masked_attention_kernel(const T* __restrict__ q, long ldq, KvSou
   const int nA = (chunk > 0) ? 0 : min(keep, lo);
   const int total = nA + (pi - lo + 1);
   float* qs = sm + wib * D;
+  scale *= query_temperature(pi, ex.temp_coef, ex.temp_every);
   for (int i = lane; i < D; i += 32) qs[i] = ldf(q + tok * ldq + h * D + i) * scale;
   __syncwarp();
   float m = -INFINITY, l = 0.f, acc[ATT_MAXV];
@@ -517,6 +639,8 @@ masked_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long ldq, const
   const int r0 = t0 + warp * 16 + gid, r1 = r0 + 8;                    // this lane's two query rows
   const int pi0 = p0 + r0, pi1 = p0 + r1;                               // their positions
   const int lo0 = mask_floor(pi0, window, chunk), lo1 = mask_floor(pi1, window, chunk);
+  const float scale0 = scale * query_temperature(pi0, ex.temp_coef, ex.temp_every);
+  const float scale1 = scale * query_temperature(pi1, ex.temp_coef, ex.temp_every);
   uint32_t qf[D / 16][4];
 #pragma unroll
   for (int kk = 0; kk < D / 16; ++kk) {
@@ -608,7 +732,7 @@ masked_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long ldq, const
       for (int j = 0; j < 8; ++j) {
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-          float sv = sacc[j][c] * scale;
+          float sv = sacc[j][c] * (c < 2 ? scale0 : scale1);
           if (capped) sv = soft_capped(sv, ex.softcap, inv_cap);
           sacc[j][c] = sv;
           if (c < 2) mx0 = fmaxf(mx0, sv); else mx1 = fmaxf(mx1, sv);
@@ -623,7 +747,7 @@ masked_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long ldq, const
           const int pj = row < ns ? row : cs + row - ns;
           const int pi = c < 2 ? pi0 : pi1, lo = c < 2 ? lo0 : lo1;
           const bool valid = row < rlim && pj <= pi && (phaseA || pj >= lo || pj < keep);
-          float sv = sacc[j][c] * scale;
+          float sv = sacc[j][c] * (c < 2 ? scale0 : scale1);
           if (capped) sv = soft_capped(sv, ex.softcap, inv_cap);
           if (!valid) sv = -INFINITY;
           sacc[j][c] = sv;
@@ -726,17 +850,20 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 ring_decode_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ ring, const T* __restrict__ first, int L, int nfirst,
                    const int* __restrict__ slots, const int* __restrict__ past, float* __restrict__ part, int H, int G, int D, int V,
-                   int window, int chunk, int keep, float scale, int splits, int vec, float softcap) {
+                   int window, int chunk, int keep, float scale, int splits, int vec, AttnExtra ex, const int* __restrict__ table,
+                   int max_pages, int page) {       // table given: `ring` is the pool of pages, L and nfirst are not used
   extern __shared__ float sm[];
+  const float softcap = ex.softcap;
   const int b = blockIdx.x, g = blockIdx.y, sp = blockIdx.z;
   const int R = H / G, C = G * (D + V), KC = G * D;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   float* qs = sm;                                   // [R][D] scaled queries
   float* red = sm + R * D;                          // [4 warps][R][V + 2]
-  for (int i = threadIdx.x; i < R * D; i += blockDim.x) qs[i] = ldf(q + (long)b * ldq + (long)g * R * D + i) * scale;
-  __syncthreads();
   const int pi = past[b];
   const long slot = slots[b];
+  scale *= query_temperature(pi, ex.temp_coef, ex.temp_every);
+  for (int i = threadIdx.x; i < R * D; i += blockDim.x) qs[i] = ldf(q + (long)b * ldq + (long)g * R * D + i) * scale;
+  __syncthreads();
   const int lo = mask_floor(pi, window, chunk);
   const int nA = chunk > 0 ? 0 : min(keep, lo);
   const int total = nA + (pi - lo + 1);
@@ -757,7 +884,9 @@ ring_decode_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ ring
     const T* vp = nullptr;
     if (mine < v1) {
       const int pj = mine < nA ? mine : lo + mine - nA;
-      const T* base = pj < nfirst ? first + (slot * nfirst + pj) * C : ring + (slot * L + pj % L) * C;
+      const T* base;
+      if (table) base = ring + ((long)table[slot * max_pages + pj / page] * page + pj % page) * C;
+      else base = pj < nfirst ? first + (slot * nfirst + pj) * C : ring + (slot * L + pj % L) * C;
       const T* kp = base + g * D;
       vp = base + KC + g * V;
 #pragma unroll
@@ -1157,6 +1286,30 @@ int lbk_qk_prepare(void* q, long ldq, void* k, long ldk, const void* qw, const v
   LAUNCH_END();
 }
 
+// keys and values to ring [*, L, C] (table null) or pool [*, page, C] when `base` is given; unit0: neither norm nor rotation -> only
+// keys and values are visited
+int lbk_heads_prepare(void* q, long ldq, void* k, long ldk, const void* v, long ldv, const void* qn, const void* kn, const float* freq,
+                      int half, int pairs, float eps, void* base, int L, const int* table, int max_pages, int page, const int* tok_seq,
+                      const int* seq_off, const int* slots, const int* past, long tokens, int H, int G, int D, int V, int dtype,
+                      cudaStream_t s) {
+  if (tokens == 0) return 0;
+  if (D > QK_MAXD || V > QK_MAXD || 2 * half > D || (base && !table && L < 1) || (table && (!base || page < 1))) return -1;
+  const int unit0 = (qn || half) ? 0 : H, units = base ? H + 2 * G : H + G;
+  if (unit0 >= units || (unit0 && !base)) return 0;
+  const int per = tokens * (units - unit0) <= 148 * 16 ? 1 : 8;
+  const long warps = tokens * ((units - unit0 + per - 1) / per);
+  const CacheRows cr{base, table, L, max_pages, page, G * (D + V), G * D};
+  const int esz = dtype ? 2 : 4;
+  auto al = [&](const void* p) { return ((uintptr_t)p % (4 * esz)) == 0; };
+  const bool vec = (pairs || !half) && D % 4 == 0 && V % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ldv % 4 == 0 && al(q) && al(k) &&
+                   al(v) && al(qn) && al(kn) && al(base);
+#define HP(TT, VV) heads_prepare_kernel<TT, VV><<<(unsigned)((warps + 3) / 4), 128, 0, s>>>((TT*)q, ldq, (TT*)k, ldk, (const TT*)v, ldv, (const TT*)qn, \
+    (const TT*)kn, freq, half, pairs, eps, cr, tok_seq, seq_off, slots, past, tokens, H, G, D, V, unit0, units, per)
+  if (dtype) { if (vec) HP(bf16, true); else HP(bf16, false); } else { if (vec) HP(float, true); else HP(float, false); }
+#undef HP
+  LAUNCH_END();
+}
+
 int lbk_kv_write(void* ring, void* first, const void* knew, const void* vnew, long ldn, const int* tok_seq, const int* seq_off,
                  const int* slots, const int* past, long tokens, int KC, int VC, int L, int nfirst, int dtype, cudaStream_t s) {
   if (tokens == 0) return 0;
@@ -1182,11 +1335,12 @@ int lbk_masked_attention(const void* q, long ldq, const void* kbase, const void*
                          int L, int nfirst, const int* ext_off, const int* nsink, const int* cstart, const int* slots,
                          const void* gate, long ldg, const int* tok_seq, const int* seq_off, const int* past, void* y, long ldy,
                          long tokens, int H, int G, int D, int V, int window, int chunk, int keep, float scale, float softcap,
-                         int sink, int gate_wide, float out_scale, int dtype, cudaStream_t s) {
+                         int sink, int gate_wide, float out_scale, float temp_coef, float temp_every, const void* pool, const int* table, int max_pages,
+                         int page, int dtype, cudaStream_t s) {
   if (tokens == 0) return 0;
-  const AttnExtra ex{softcap, out_scale, sink, gate_wide};
+  const AttnExtra ex{softcap, out_scale, sink, gate_wide, temp_coef, temp_every};
   if (V > 32 * ATT_MAXV || G <= 0 || H % G) return -1;
-  KvSource src{kbase, vbase, ldkv, ring, first, L, nfirst, G * (D + V), G * D, ext_off, nsink, cstart, slots};
+  KvSource src{kbase, vbase, ldkv, ring, first, L, nfirst, G * (D + V), G * D, pool, table, max_pages, page, ext_off, nsink, cstart, slots};
   const int warps = 4;
   const long nwarps = tokens * H;
   const unsigned grid = (unsigned)((nwarps + warps - 1) / warps);
@@ -1248,10 +1402,10 @@ int lbk_masked_attention_mma(const void* q, long ldq, const void* kbase, const v
                              const int* nsink, const int* cstart, const void* gate, long ldg, const int* qt_seq, const int* qt_start,
                              int n_qtiles, const int* seq_off, const int* past, void* y, long ldy, int H, int G, int D, int V,
                              int window, int chunk, int keep, float scale, float softcap, int sink, int gate_wide, float out_scale,
-                             cudaStream_t s) {
+                             float temp_coef, float temp_every, cudaStream_t s) {
   if (n_qtiles == 0) return 0;
   if (D != V || G <= 0 || H % G) return -1;
-  const AttnExtra ex{softcap, out_scale, sink, gate_wide};
+  const AttnExtra ex{softcap, out_scale, sink, gate_wide, temp_coef, temp_every};
   const dim3 grid((unsigned)n_qtiles, (unsigned)H);
 #define MMA_CASE(DD) case DD: { \
     constexpr int smem = 2 * 64 * (2 * DD + 16) * 2; \
@@ -1270,10 +1424,10 @@ int lbk_masked_attention_mma(const void* q, long ldq, const void* kbase, const v
 
 int lbk_ring_decode(const void* q, long ldq, const void* ring, const void* first, int L, int nfirst, const int* slots, const int* past,
                     const void* gate, long ldg, void* y, long ldy, float* part, int B, int H, int G, int D, int V, int window,
-                    int chunk, int keep, float scale, int splits, float softcap, int sink, int gate_wide, float out_scale, int dtype,
-                    cudaStream_t s) {
+                    int chunk, int keep, float scale, int splits, float softcap, int sink, int gate_wide, float out_scale, float temp_coef,
+                    float temp_every, const int* table, int max_pages, int page, int dtype, cudaStream_t s) {
   if (B == 0) return 0;
-  const AttnExtra ex{softcap, out_scale, sink, gate_wide};
+  const AttnExtra ex{softcap, out_scale, sink, gate_wide, temp_coef, temp_every};
   if (G <= 0 || H % G || H / G > DEC_MAXR || V > 32 * DEC_MAXVL || splits < 1) return -1;
   const int R = H / G;
   const size_t smem = ((size_t)R * D + 4 * (size_t)R * (V + 2)) * sizeof(float);
@@ -1283,12 +1437,12 @@ int lbk_ring_decode(const void* q, long ldq, const void* ring, const void* first
   if (dtype) {
     const int vec = (D % 8 == 0 && C % 8 == 0 && ((uintptr_t)ring & 15) == 0 && ((uintptr_t)first & 15) == 0) ? 1 : 0;
     ring_decode_kernel<bf16><<<grid, 128, smem, s>>>((const bf16*)q, ldq, (const bf16*)ring, (const bf16*)first, L, nfirst, slots, past,
-                                                     part, H, G, D, V, window, chunk, keep, scale, splits, vec, softcap);
+                                                     part, H, G, D, V, window, chunk, keep, scale, splits, vec, ex, table, max_pages, page);
     ring_decode_merge_kernel<bf16><<<dim3((unsigned)B, (unsigned)H), 64, 0, s>>>(part, (const bf16*)gate, ldg, (bf16*)y, ldy, H, V, splits, ex);
   } else {
     const int vec = (D % 8 == 0 && C % 4 == 0 && ((uintptr_t)ring & 15) == 0 && ((uintptr_t)first & 15) == 0) ? 1 : 0;
     ring_decode_kernel<float><<<grid, 128, smem, s>>>((const float*)q, ldq, (const float*)ring, (const float*)first, L, nfirst, slots,
-                                                      past, part, H, G, D, V, window, chunk, keep, scale, splits, vec, softcap);
+                                                      past, part, H, G, D, V, window, chunk, keep, scale, splits, vec, ex, table, max_pages, page);
     ring_decode_merge_kernel<float><<<dim3((unsigned)B, (unsigned)H), 64, 0, s>>>(part, (const float*)gate, ldg, (float*)y, ldy, H, V, splits, ex);
   }
   LAUNCH_END();

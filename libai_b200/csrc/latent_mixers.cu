@@ -136,10 +136,11 @@ latent_prepare_kernel(const T* __restrict__ dkv, long ldk, const T* __restrict__
   for (int i = C + R + lane; i < CS; i += 32) { stf(row + i, 0.f); if (out) stf(out + i, 0.f); }
 }
 
-// ext[e] = the cache row of position e - ext_off[b] of sequence b = ext_seq[e]; 16 bytes per thread
-__global__ void latent_pages_gather_kernel(const uint4* __restrict__ pool, const int* __restrict__ table, int max_pages, int page_size,
+// ext[e] = the cache row of position e - ext_off[b] of sequence b = ext_seq[e]; one unit U per thread (16 bytes where the rows allow it)
+template <typename U>
+__global__ void latent_pages_gather_kernel(const U* __restrict__ pool, const int* __restrict__ table, int max_pages, int page_size,
                                            const int* __restrict__ ext_seq, const int* __restrict__ ext_off, const int* __restrict__ slots,
-                                           uint4* __restrict__ ext, long rows, int vecs) {
+                                           U* __restrict__ ext, long rows, int vecs) {
   const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= rows * vecs) return;
   const long e = i / vecs;
@@ -859,10 +860,12 @@ int lbl_latent_pages_gather(const void* pool, const int* table, int max_pages, i
                             const int* slots, void* ext, long rows, int CS, int dtype, cudaStream_t s) {
   if (rows == 0) return 0;
   const long bytes = (long)CS * (dtype ? 2 : 4);
-  if (bytes % 16 != 0 || ((uintptr_t)pool & 15) != 0 || ((uintptr_t)ext & 15) != 0) return -1;
-  const int vecs = (int)(bytes / 16);
-  latent_pages_gather_kernel<<<(unsigned)((rows * vecs + 255) / 256), 256, 0, s>>>((const uint4*)pool, table, max_pages, page_size, ext_seq, ext_off,
-                                                                                   slots, (uint4*)ext, rows, vecs);
+  const bool wide = bytes % 16 == 0 && ((uintptr_t)pool & 15) == 0 && ((uintptr_t)ext & 15) == 0;
+  const int unit = wide ? 16 : (dtype ? 2 : 4), vecs = (int)(bytes / unit);
+  const unsigned grid = (unsigned)((rows * vecs + 255) / 256);
+#define PGA(U) latent_pages_gather_kernel<U><<<grid, 256, 0, s>>>((const U*)pool, table, max_pages, page_size, ext_seq, ext_off, slots, (U*)ext, rows, vecs)
+  if (unit == 16) PGA(uint4); else if (unit == 2) PGA(uint16_t); else PGA(uint32_t);
+#undef PGA
   LAUNCH_END();
 }
 

@@ -17,6 +17,15 @@ int lbl_decay_scan(const void* q, long ldq, const void* k, long ldk, const void*
                    long ldz, const float* zb, const float* lower, float inv_tau, float q_scale, float k_scale, int act, float* S,
                    const int* seq_off, const int* slots, const int* past, float* out, int B, int H, int D, int V, int dtype,
                    cudaStream_t s);
+int lbl_memory_gates(const float* z, long ldz, int foff, const float* zb, float cap, float* mx, const int* seq_off, const int* slots,
+                     const int* past, float* gates, long tokens, int B, int H, cudaStream_t s);
+int lbl_memory_scan(const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, const float* gates, float q_scale, float* S,
+                    float* Z, float* ztmp, const int* seq_off, const int* slots, const int* past, float* out, long tokens, int B, int H, int D, int V,
+                    int dtype, cudaStream_t s);
+int lbl_memory_step(const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, const float* z, long ldz, int foff,
+                    const float* zb, float cap, float q_scale, float* S, float* Z, float* mx, const int* slots, const int* past, const void* w,
+                    const void* gate, long ldg, float eps, float out_scale, void* y, long ldy, int B, int H, int D, int V, int dtype,
+                    cudaStream_t s);
 int lbl_gated_norm(const float* o, const void* gate, long ldg, const void* w, float eps, int act, float out_scale, void* y, long ldy,
                    long rows, int H, int V, int per_head, int dtype, cudaStream_t s);
 }
@@ -121,7 +130,7 @@ void decay_scan(const Tensor& q, const Tensor& k, const Tensor& v, const OptT& d
 }
 
 void gated_norm(const Tensor& o, const OptT& gate_opt, const OptT& w, double eps, int64_t act, double out_scale, Tensor y, int64_t H, int64_t V,
-                bool per_head) {
+                bool per_head, bool wide) {
   TORCH_CHECK(has(gate_opt) || act == 2, "gated_norm: a gate, or act 2 (none)");
   const Tensor& gate = has(gate_opt) ? *gate_opt : y;      // act 2 reads no gate
   rows2d(gate, "gated_norm gate"); rows2d(y, "gated_norm y");
@@ -129,12 +138,64 @@ void gated_norm(const Tensor& o, const OptT& gate_opt, const OptT& w, double eps
   TORCH_CHECK(gate.size(1) == H * V && gate.size(0) == y.size(0) && y.size(1) == H * V && code(gate) == code(y), "gated_norm: shapes");
   const void* wp = nullptr;
   if (has(w)) {
-    TORCH_CHECK(w->is_cuda() && w->is_contiguous() && w->numel() == (per_head ? V : H * V) && code(*w) == code(y), "gated_norm: weight");
+    TORCH_CHECK(w->is_cuda() && w->is_contiguous() && w->numel() == (per_head && !wide ? V : H * V) && code(*w) == code(y), "gated_norm: weight");
     wp = w->data_ptr();
   }
   c10::cuda::CUDAGuard guard(o.device());
   check(lbl_gated_norm(o.data_ptr<float>(), gate.data_ptr(), gate.stride(0), wp, (float)eps, (int)act, (float)out_scale, y.data_ptr(),
-                       y.stride(0), y.size(0), (int)H, (int)V, per_head ? 1 : 0, code(y), cur_stream()), "gated_norm");
+                       y.stride(0), y.size(0), (int)H, (int)V, per_head ? (wide ? 2 : 1) : 0, code(y), cur_stream()), "gated_norm");
+}
+
+struct MemoryShape { int H, D, V; };
+MemoryShape memory_state(const Tensor& S, const Tensor& Z, const Tensor& mx) {
+  TORCH_CHECK(S.is_cuda() && S.dim() == 4 && S.is_contiguous() && S.scalar_type() == at::kFloat, "memory: S must be fp32 [slots, H, D, V]");
+  TORCH_CHECK(Z.is_cuda() && Z.dim() == 3 && Z.is_contiguous() && Z.scalar_type() == at::kFloat && Z.size(0) == S.size(0) && Z.size(1) == S.size(1) &&
+              Z.size(2) == S.size(2) && mx.is_cuda() && mx.dim() == 2 && mx.is_contiguous() && mx.scalar_type() == at::kFloat &&
+              mx.size(0) == S.size(0) && mx.size(1) == S.size(1), "memory: key sums fp32 [slots, H, D] and maxima fp32 [slots, H]");
+  return {(int)S.size(1), (int)S.size(2), (int)S.size(3)};
+}
+void memory_operands(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& z, const Tensor& zb, int64_t foff, const MemoryShape& m) {
+  rows2d(q, "memory q"); rows2d(k, "memory k"); rows2d(v, "memory v"); rows2d(z, "memory z");
+  TORCH_CHECK(q.size(1) == (long)m.H * m.D && k.size(1) == (long)m.H * m.D && v.size(1) == (long)m.H * m.V && k.size(0) == q.size(0) &&
+              v.size(0) == q.size(0) && code(q) == code(k) && code(q) == code(v), "memory: q, k [tokens, H*D], v [tokens, H*V] of one dtype");
+  TORCH_CHECK(z.scalar_type() == at::kFloat && z.size(0) == q.size(0) && foff >= m.H && z.size(1) >= foff + m.H, "memory: gate logits fp32 [tokens, >= foff + H]");
+  f32(zb, z.size(1), "memory: gate biases");
+}
+
+// gate logits of a step: columns 0..H-1 input gates, foff..foff+H-1 forget gates; out fp32 [tokens, H*V]
+void memory_scan(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& z, const Tensor& zb, int64_t foff, double cap, double q_scale,
+                 Tensor S, Tensor Z, Tensor mx, const Tensor& seq_off, const Tensor& slots, const Tensor& past, Tensor out) {
+  const MemoryShape m = memory_state(S, Z, mx);
+  memory_operands(q, k, v, z, zb, foff, m);
+  TORCH_CHECK(out.is_cuda() && out.scalar_type() == at::kFloat && out.is_contiguous() && out.dim() == 2 && out.size(1) == (long)m.H * m.V &&
+              out.size(0) == q.size(0), "memory_scan: out must be fp32 [tokens, H*V]");
+  c10::cuda::CUDAGuard guard(q.device());
+  const int64_t tokens = q.size(0);
+  const int B = (int)slots.numel();
+  Tensor gates = at::empty({m.H, 3, tokens}, z.options()), ztmp = at::empty({B, m.H, m.D}, z.options());
+  check(lbl_memory_gates(z.data_ptr<float>(), z.stride(0), (int)foff, zb.data_ptr<float>(), (float)cap, mx.data_ptr<float>(), meta(seq_off), meta(slots),
+                         meta(past), gates.data_ptr<float>(), tokens, B, m.H, cur_stream()), "memory_gates");
+  check(lbl_memory_scan(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), gates.data_ptr<float>(), (float)q_scale,
+                        S.data_ptr<float>(), Z.data_ptr<float>(), ztmp.data_ptr<float>(), meta(seq_off), meta(slots), meta(past), out.data_ptr<float>(), tokens, B, m.H, m.D,
+                        m.V, code(q), cur_stream()), "memory_scan");
+}
+
+// one token per sequence, through to the gated, normed read-out y [tokens, H*V]
+void memory_step(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& z, const Tensor& zb, int64_t foff, double cap, double q_scale,
+                 Tensor S, Tensor Z, Tensor mx, const Tensor& slots, const Tensor& past, const OptT& w, const OptT& gate, double eps,
+                 double out_scale, Tensor y) {
+  const MemoryShape m = memory_state(S, Z, mx);
+  memory_operands(q, k, v, z, zb, foff, m);
+  rows2d(y, "memory_step y");
+  TORCH_CHECK(q.size(0) == slots.numel() && y.size(0) == q.size(0) && y.size(1) == (long)m.H * m.V && code(y) == code(q), "memory_step: one token per sequence");
+  long ldg = 0;
+  if (has(gate)) { rows2d(*gate, "memory_step gate"); TORCH_CHECK(gate->size(0) == y.size(0) && gate->size(1) == y.size(1) && code(*gate) == code(y), "memory_step: gate [tokens, H*V]"); ldg = gate->stride(0); }
+  if (has(w)) TORCH_CHECK(w->is_cuda() && w->is_contiguous() && w->numel() == (long)m.H * m.V && code(*w) == code(y), "memory_step: weight [H*V]");
+  c10::cuda::CUDAGuard guard(q.device());
+  check(lbl_memory_step(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), z.data_ptr<float>(), z.stride(0), (int)foff,
+                        zb.data_ptr<float>(), (float)cap, (float)q_scale, S.data_ptr<float>(), Z.data_ptr<float>(), mx.data_ptr<float>(), meta(slots),
+                        meta(past), has(w) ? w->data_ptr() : nullptr, has(gate) ? gate->data_ptr() : nullptr, ldg, (float)eps, (float)out_scale,
+                        y.data_ptr(), y.stride(0), (int)slots.numel(), m.H, m.D, m.V, code(q), cur_stream()), "memory_step");
 }
 }  // namespace
 
@@ -142,5 +203,7 @@ TORCH_LIBRARY(libai_b200_lin, m) {
   m.def("embed_bigram(Tensor table, Tensor bigram, Tensor ids, Tensor(a!) last, Tensor tok_seq, Tensor seq_off, Tensor slots, Tensor past, float scale, int mul_prev, int mul_cur, int buckets, Tensor(b!) x) -> ()", &embed_bigram);
   m.def("hc_step(Tensor(a!) x, Tensor? y, Tensor? pos, Tensor? cw, Tensor? mix, Tensor? outw, Tensor? inw, Tensor? w, float eps, Tensor(b!)? h) -> ()", &hc_step);
   m.def("decay_scan(Tensor q, Tensor k, Tensor v, Tensor? decay, Tensor? z, Tensor? zb, float inv_tau, float q_scale, float k_scale, int act, Tensor(a!) S, Tensor seq_off, Tensor slots, Tensor past, Tensor(b!) out, Tensor? lower=None) -> ()", &decay_scan);
-  m.def("gated_norm(Tensor o, Tensor? gate, Tensor? w, float eps, int act, float out_scale, Tensor(a!) y, int H, int V, bool per_head) -> ()", &gated_norm);
+  m.def("gated_norm(Tensor o, Tensor? gate, Tensor? w, float eps, int act, float out_scale, Tensor(a!) y, int H, int V, bool per_head, bool wide=False) -> ()", &gated_norm);
+  m.def("memory_scan(Tensor q, Tensor k, Tensor v, Tensor z, Tensor zb, int foff, float cap, float q_scale, Tensor(a!) S, Tensor(b!) Z, Tensor(c!) mx, Tensor seq_off, Tensor slots, Tensor past, Tensor(d!) out) -> ()", &memory_scan);
+  m.def("memory_step(Tensor q, Tensor k, Tensor v, Tensor z, Tensor zb, int foff, float cap, float q_scale, Tensor(a!) S, Tensor(b!) Z, Tensor(c!) mx, Tensor slots, Tensor past, Tensor? w, Tensor? gate, float eps, float out_scale, Tensor(d!) y) -> ()", &memory_step);
 }

@@ -271,6 +271,10 @@ __global__ void hc_step_vec_kernel(float* __restrict__ x, long rows, int n, int 
 // a padded offset: 16-byte loads without bank conflicts) with activations, scales and decays applied during staging; the
 // global loads of the next group are issued before the serial walk over the current one and land in the other buffer
 // afterwards.
+//
+// MEM: the matrix memory with exponential gates (see memory_gates_kernel below).  The decay is one number per head and token,
+// the key is multiplied by the token's write weight, a second state z [slots, H, D] sums the weighted keys without values, and the
+// read-out is divided by max(|z q|, floor) + 1e-6.  gates [H][3][tokens]: decay, write weight, floor.
 // ------------------------------------------------------------------------------------------------------------------
 constexpr int SCAN_CT = 16, SCAN_NC = 8;
 
@@ -294,27 +298,32 @@ template <> __device__ __forceinline__ void ldn<bf16, 8>(const bf16* p, float (&
   for (int i = 0; i < 4; ++i) { f[2 * i] = __low2float(h2[i]); f[2 * i + 1] = __high2float(h2[i]); }
 }
 
-template <typename T, int DPT>
+template <typename T, int DPT, bool MEM>
 __global__ void __launch_bounds__(256, 1)
 decay_scan_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, long ldk, const T* __restrict__ v, long ldv,
                   const float* __restrict__ decay, const float* __restrict__ z, long ldz, const float* __restrict__ zb,
                   const float* __restrict__ lower, float inv_tau, float q_scale, float k_scale, int act, float* __restrict__ S, const int* __restrict__ seq_off,
                   const int* __restrict__ slots, const int* __restrict__ past, float* __restrict__ out, int H, int D, int V, int R,
-                  int VT, int CT, int vec) {
+                  int VT, int CT, int vec, const float* __restrict__ gates, float* Z, float* ztmp, long tokens) {
   extern __shared__ __align__(16) float sm[];
   constexpr int NC = SCAN_NC, PS = DPT == 8 ? 12 : 4;   // padded stride of one lane's rows
   const int b = blockIdx.x / H, h = blockIdx.x % H;
   const int j0 = blockIdx.y * VT;
   const int Dp = R * PS;                        // floats per staged token
   const bool chan = z != nullptr;
-  const int buf_floats = CT * (Dp * (chan ? 3 : 2) + VT);
+  const int buf_floats = CT * (Dp * (chan ? 3 : 2) + VT + (MEM ? 4 : 0));
   const int tid = threadIdx.x, nth = blockDim.x;
   const int r = tid % R, grp = tid / R;         // lane within the column group, column group
   const int jc = j0 + grp * NC;                 // first of this thread's 8 columns
   const bool grp_ok = grp * NC < VT;
   const int n = seq_off[b + 1] - seq_off[b];
   const long tok0 = seq_off[b];
-  const float g0 = chan ? 1.f : decay[h];
+  const float g0 = (MEM || chan) ? 1.f : decay[h];
+  const float* gt = MEM ? gates + (long)h * 3 * tokens : nullptr;
+  float* Zg = MEM ? Z + ((long)slots[b] * H + h) * D : nullptr;
+  float nz[DPT];
+#pragma unroll
+  for (int d = 0; d < DPT; ++d) nz[d] = (MEM && past[b] > 0 && r * DPT + d < D) ? Zg[r * DPT + d] : 0.f;
   float* Sg = S + ((long)slots[b] * H + h) * (long)D * V;
   float s[DPT][NC];
 #pragma unroll
@@ -326,13 +335,17 @@ decay_scan_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, lo
   // staging work of this thread: one (token, lane chunk) of q / k / decays and one (token, column group) of v per group of CT
   // tokens (the launcher picks CT so that both fit the block)
   const int qk_items = CT * R, v_items = CT * (VT / NC);
-  float rk[DPT], rq[DPT], rg[DPT], rl[DPT], rv[NC];
+  float rk[DPT], rq[DPT], rg[DPT], rl[DPT], rv[NC], rw = 1.f, ra = 1.f, re = 1.f;
   auto fetch = [&](int c0) {                    // global loads of the group that starts at token c0, into registers
     const int ct = min(CT, n - c0);
     if (tid < qk_items) {
       const int t = tid / R, rr = tid - t * R;
       const long row = tok0 + c0 + t;
       const int i0 = rr * DPT;
+      if (MEM) {
+        rw = t < ct ? gt[tokens + row] : 0.f;
+        if (rr == 0) { ra = t < ct ? gt[row] : 1.f; re = t < ct ? gt[2 * tokens + row] : 1.f; }
+      }
       if (t < ct && vec && i0 + DPT <= D) {
         if (!lower) ldn<T, DPT>(k + row * ldk + h * D + i0, rk);
         else ldn<float, DPT>(lower + h * D + i0, rl);
@@ -383,6 +396,7 @@ decay_scan_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, lo
           kv = 1.f - go[d];
         }
         ko[d] = kv * k_scale; qo[d] = qv * q_scale;
+        if (MEM) ko[d] *= rw;
       }
 #pragma unroll
       for (int d4 = 0; d4 < DPT / 4; ++d4) {
@@ -390,6 +404,7 @@ decay_scan_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, lo
         reinterpret_cast<float4*>(sq + t * Dp + rr * PS)[d4] = make_float4(qo[4 * d4], qo[4 * d4 + 1], qo[4 * d4 + 2], qo[4 * d4 + 3]);
         if (chan) reinterpret_cast<float4*>(sg + t * Dp + rr * PS)[d4] = make_float4(go[4 * d4], go[4 * d4 + 1], go[4 * d4 + 2], go[4 * d4 + 3]);
       }
+      if (MEM && rr == 0) { float* sgate = sv + CT * VT; sgate[2 * t] = ra; sgate[2 * t + 1] = re; }
     }
     if (tid < v_items) {
       float vo[NC];
@@ -411,6 +426,7 @@ decay_scan_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, lo
     const float* buf = sm + cur * buf_floats;
     const float* sk = buf + r * PS; const float* sq = sk + CT * Dp; const float* sg = sq + CT * Dp;
     const float* sv = buf + CT * Dp * (chan ? 3 : 2) + (grp_ok ? grp * NC : 0);
+    const float* sgate = buf + CT * Dp * (chan ? 3 : 2) + CT * VT;
     float* orow = out + (tok0 + c0) * (long)(H * V) + h * V;
     // every thread walks the tokens (lanes of idle column groups included: the shuffles below name the whole warp)
 #pragma unroll 2
@@ -418,12 +434,14 @@ decay_scan_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, lo
       const float4 va = reinterpret_cast<const float4*>(sv)[0], vb = reinterpret_cast<const float4*>(sv)[1];
       const float vt[NC] = {va.x, va.y, va.z, va.w, vb.x, vb.y, vb.z, vb.w};
       float o[NC];
+      float zq = 0.f, div = 1.f;
+      const float gm = MEM ? sgate[2 * t] : g0;
 #pragma unroll
       for (int c = 0; c < NC; ++c) o[c] = 0.f;
 #pragma unroll
       for (int d4 = 0; d4 < DPT / 4; ++d4) {
         const float4 kx = reinterpret_cast<const float4*>(sk)[d4], qx = reinterpret_cast<const float4*>(sq)[d4];
-        float4 gx = make_float4(g0, g0, g0, g0);
+        float4 gx = make_float4(gm, gm, gm, gm);
         if (chan) gx = reinterpret_cast<const float4*>(sg)[d4];
         const float kk[4] = {kx.x, kx.y, kx.z, kx.w}, qq[4] = {qx.x, qx.y, qx.z, qx.w}, gg[4] = {gx.x, gx.y, gx.z, gx.w};
 #pragma unroll
@@ -433,7 +451,12 @@ decay_scan_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, lo
             s[4 * d4 + e][c] = s[4 * d4 + e][c] * gg[e] + kk[e] * vt[c];
             o[c] += s[4 * d4 + e][c] * qq[e];
           }
+          if (MEM) { nz[4 * d4 + e] = nz[4 * d4 + e] * gm + kk[e]; zq += nz[4 * d4 + e] * qq[e]; }
         }
+      }
+      if (MEM) {
+        for (int m = R >> 1; m > 0; m >>= 1) zq += __shfl_xor_sync(0xffffffffu, zq, m);
+        div = 1.f / (fmaxf(fabsf(zq), sgate[2 * t + 1]) + 1e-6f);
       }
       if (R >= 8) {
         // transposing butterfly: after three rounds a lane holds, for one column, the sum over its 8 neighbouring lanes
@@ -446,7 +469,7 @@ decay_scan_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, lo
         float w = (b2 ? bq[1] : bq[0]) + __shfl_xor_sync(0xffffffffu, b2 ? bq[0] : bq[1], 4);
         for (int m = 8; m < R; m <<= 1) w += __shfl_xor_sync(0xffffffffu, w, m);
         const int col = jc + (b0 ? 4 : 0) + (b1 ? 2 : 0) + (b2 ? 1 : 0);
-        if (r < 8 && grp_ok && col < V) orow[col] = w;
+        if (r < 8 && grp_ok && col < V) orow[col] = MEM ? w * div : w;
       } else {
         for (int m = R >> 1; m > 0; m >>= 1) {
 #pragma unroll
@@ -454,7 +477,7 @@ decay_scan_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, lo
         }
         if (r == 0 && grp_ok) {
 #pragma unroll
-          for (int c = 0; c < NC; ++c) if (jc + c < V) orow[jc + c] = o[c];
+          for (int c = 0; c < NC; ++c) if (jc + c < V) orow[jc + c] = MEM ? o[c] * div : o[c];
         }
       }
     }
@@ -468,23 +491,156 @@ decay_scan_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, lo
       const int i = r * DPT + d;
 #pragma unroll
       for (int c = 0; c < NC; ++c) if (i < D && jc + c < V) Sg[(long)i * V + jc + c] = s[d][c];
+      // with several column tiles a block may start after this one ended, and must still read the old z
+      if (MEM && grp == 0 && blockIdx.y == 0 && i < D) (gridDim.y > 1 ? ztmp + (long)blockIdx.x * D : Zg)[i] = nz[d];
     }
   }
 }
 
 // ------------------------------------------------------------------------------------------------------------------
+// Matrix memory with exponential gates (the mLSTM cell of Beck et al., "xLSTM: Extended Long Short-Term Memory", 2024).  Per head, from the
+// fp32 logits zi, zf (+ their biases): i = cap tanh(zi / cap) and f = log sigmoid(cap tanh(zf / cap)) are the log gates, a running
+// maximum (0 at the start of a sequence) keeps the state in range,
+//   m_t = max(f + m_(t-1), i),   decay = exp(f + m_(t-1) - m_t),   write = exp(i - m_t),   floor = exp(-m_t),
+//   S <- decay S + write k v^T,   z <- decay z + write k,   o = S^T q / (max(|z q|, floor) + 1e-6).
+// memory_gates_kernel: one warp per (sequence, head) turns the logits of the step into gates [H][3][tokens] = decay, write, floor, 32 tokens
+// at a time: with F_t = sum of f over the group, m_t = max(F_t + m_in, max_s (i_s + F_t - F_s)) is a scan of (f, i) pairs under
+// (F1 + F2, max(M1 + F2, M2)).  mx [slots, H] holds the running maximum between steps.
+// ------------------------------------------------------------------------------------------------------------------
+__device__ __forceinline__ void memory_log_gates(float zi, float zf, float cap, float& li, float& lf) {
+  li = cap * tanhf(zi / cap);
+  lf = logsigmoidf_(cap * tanhf(zf / cap));
+}
+
+__global__ void memory_keysum_kernel(const float* __restrict__ ztmp, float* __restrict__ Z, const int* __restrict__ slots, int H, int D) {
+  const int b = blockIdx.x / H, h = blockIdx.x - b * H;
+  for (int i = threadIdx.x; i < D; i += blockDim.x) Z[((long)slots[b] * H + h) * D + i] = ztmp[(long)blockIdx.x * D + i];
+}
+
+__global__ void memory_gates_kernel(const float* __restrict__ z, long ldz, int foff, const float* __restrict__ zb, float cap,
+                                    float* __restrict__ mx, const int* __restrict__ seq_off, const int* __restrict__ slots,
+                                    const int* __restrict__ past, float* __restrict__ gates, long tokens, int B, int H) {
+  const int wid = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (wid >= B * H) return;
+  const int b = wid / H, h = wid - b * H;
+  const long tok0 = seq_off[b];
+  const int n = seq_off[b + 1] - seq_off[b];
+  float* mslot = mx + (long)slots[b] * H + h;
+  float m = past[b] > 0 ? *mslot : 0.f;
+  const float bi = zb[h], bf = zb[foff + h];
+  float* g0 = gates + (long)h * 3 * tokens + tok0;
+  for (int t0 = 0; t0 < n; t0 += 32) {
+    const int t = t0 + lane;
+    float li = -INFINITY, lf = 0.f;               // beyond the end: the maximum stays
+    if (t < n) memory_log_gates(z[(tok0 + t) * ldz + h] + bi, z[(tok0 + t) * ldz + foff + h] + bf, cap, li, lf);
+    float F = lf, M = li;
+#pragma unroll
+    for (int d = 1; d < 32; d <<= 1) {
+      const float Fp = __shfl_up_sync(0xffffffffu, F, d), Mp = __shfl_up_sync(0xffffffffu, M, d);
+      if (lane >= d) { M = fmaxf(Mp + F, M); F += Fp; }
+    }
+    const float mt = fmaxf(F + m, M);
+    float mp = __shfl_up_sync(0xffffffffu, mt, 1);
+    if (lane == 0) mp = m;
+    if (t < n) {
+      g0[t] = expf(lf + mp - mt);
+      g0[tokens + t] = expf(li - mt);
+      g0[2 * tokens + t] = expf(-mt);
+    }
+    m = __shfl_sync(0xffffffffu, mt, 31);
+  }
+  if (lane == 0) *mslot = m;
+}
+
+// One token per sequence: gates, state update, read-out, per-head RMS norm, weight w [H*V] and sigmoid gate in one block per (sequence, head).
+// A thread owns NV neighbouring columns of the rows rg, rg + RG, ...; the partial read-outs meet in shared memory.
+template <typename T, int NV>
+__global__ void __launch_bounds__(512)
+memory_step_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, long ldk, const T* __restrict__ v, long ldv,
+                   const float* __restrict__ z, long ldz, int foff, const float* __restrict__ zb, float cap, float q_scale,
+                   float* __restrict__ S, float* __restrict__ Z, float* __restrict__ mx, const int* __restrict__ slots,
+                   const int* __restrict__ past, const T* __restrict__ w, const T* __restrict__ gate, long ldg, float eps, float out_scale,
+                   T* __restrict__ y, long ldy, int H, int D, int V, int RG) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float red[32];
+  const int b = blockIdx.x / H, h = blockIdx.x - b * H, tid = threadIdx.x;
+  float* ks = sm; float* qs = ks + D; float* os = qs + D;             // os [RG][V]
+  const long slot = slots[b];
+  const bool cont = past[b] > 0;
+  float* mslot = mx + slot * H + h;
+  const float m0 = cont ? *mslot : 0.f;
+  float li, lf;
+  memory_log_gates(z[b * ldz + h] + zb[h], z[b * ldz + foff + h] + zb[foff + h], cap, li, lf);
+  const float m1 = fmaxf(lf + m0, li);
+  const float dec = expf(lf + m0 - m1), put = expf(li - m1), flo = expf(-m1);
+  float* Zg = Z + (slot * H + h) * D;
+  float zq = 0.f;
+  for (int i = tid; i < D; i += blockDim.x) {
+    const float kv = ldf(k + b * ldk + h * D + i) * put, qv = ldf(q + b * ldq + h * D + i) * q_scale;
+    ks[i] = kv; qs[i] = qv;
+    const float zn = (cont ? Zg[i] : 0.f) * dec + kv;
+    Zg[i] = zn;
+    zq += zn * qv;
+  }
+  zq = block_sum(zq, red);                          // (its barriers also publish ks / qs, and every thread has read mx)
+  if (tid == 0) *mslot = m1;
+  const int VG = (V + NV - 1) / NV;
+  float* Sg = S + (slot * H + h) * (long)D * V;
+  for (int it = tid; it < VG * RG; it += blockDim.x) {
+    const int rg = it / VG, c = (it - rg * VG) * NV;
+    float vt[NV], o[NV];
+#pragma unroll
+    for (int j = 0; j < NV; ++j) { vt[j] = c + j < V ? ldf(v + b * ldv + h * V + c + j) : 0.f; o[j] = 0.f; }
+#pragma unroll 4
+    for (int i = rg; i < D; i += RG) {
+      float* p = Sg + (long)i * V + c;
+      const float kv = ks[i], qv = qs[i];
+      if (NV == 4) {
+        float4 s4 = cont ? *reinterpret_cast<const float4*>(p) : make_float4(0.f, 0.f, 0.f, 0.f);
+        s4.x = s4.x * dec + kv * vt[0]; s4.y = s4.y * dec + kv * vt[1 % NV]; s4.z = s4.z * dec + kv * vt[2 % NV]; s4.w = s4.w * dec + kv * vt[3 % NV];
+        *reinterpret_cast<float4*>(p) = s4;
+        o[0] += s4.x * qv; o[1 % NV] += s4.y * qv; o[2 % NV] += s4.z * qv; o[3 % NV] += s4.w * qv;
+      } else {
+        const float s1 = (cont ? *p : 0.f) * dec + kv * vt[0];
+        *p = s1;
+        o[0] += s1 * qv;
+      }
+    }
+#pragma unroll
+    for (int j = 0; j < NV; ++j) if (c + j < V) os[rg * V + c + j] = o[j];
+  }
+  __syncthreads();
+  const float div = 1.f / (fmaxf(fabsf(zq), flo) + 1e-6f);
+  float ss = 0.f;
+  for (int c = tid; c < V; c += blockDim.x) {
+    float o = 0.f;
+    for (int g = 0; g < RG; ++g) o += os[g * V + c];
+    o *= div;
+    os[c] = o;                                      // column c of every row group is read and written by this thread only
+    ss += o * o;
+  }
+  ss = block_sum(ss, red);
+  const float rr = out_scale / sqrtf(ss / (float)V + eps);
+  for (int c = tid; c < V; c += blockDim.x) {
+    const float ga = gate ? sigmoidf_(ldf(gate + b * ldg + h * V + c)) : 1.f;
+    stf(y + b * ldy + h * V + c, os[c] * rr * (w ? ldf(w + h * V + c) : 1.f) * ga);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------------------
 // Gated RMS norm of a read-out o [rows, H*V] (fp32):  y = o / sqrt(mean(o^2) + eps) * w * act(gate) * out_scale, the
-// mean taken over the V channels of every head (per_head = 1, w [V] shared by the heads or absent) or over the whole
+// mean taken over the V channels of every head (per_head = 1, w [V] shared by the heads or absent; per_head = 2: w [H*V]) or over the whole
 // row (per_head = 0, w [H*V] or absent); act 0: silu, 1: sigmoid, 2: no gate (the gate pointer is not read).  One warp per
 // (row, head), or one block per row.
 // ------------------------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void gated_norm_head_kernel(const float* __restrict__ o, const T* __restrict__ gate, long ldg, const T* __restrict__ w,
-                                       float eps, int act, float out_scale, T* __restrict__ y, long ldy, long rows, int H, int V, int vec) {
+                                       float eps, int act, float out_scale, T* __restrict__ y, long ldy, long rows, int H, int V, int wide, int vec) {
   const long wid = ((long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
   if (wid >= rows * H) return;
   const long tok = wid / H; const int h = (int)(wid - tok * H);
+  if (wide && w) w += h * V;                      // a weight per head and channel
   const float* orow = o + (tok * H + h) * (long)V;
   float ss = 0.f;
   if (vec) {                                     // four channels per lane and access (the second pass re-reads o from L1)
@@ -602,12 +758,13 @@ int lbl_hc_step(float* x, long rows, int n, int ns, const void* y, long ldy, int
   LAUNCH_END();
 }
 
-int lbl_decay_scan(const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, const float* decay, const float* z,
-                   long ldz, const float* zb, const float* lower, float inv_tau, float q_scale, float k_scale, int act, float* S,
-                   const int* seq_off, const int* slots, const int* past, float* out, int B, int H, int D, int V, int dtype,
-                   cudaStream_t s) {
+// gates / Z: the matrix memory's form (decay, z, lower absent)
+static int launch_scan(const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, const float* decay, const float* z,
+                       long ldz, const float* zb, const float* lower, float inv_tau, float q_scale, float k_scale, int act, float* S,
+                       const int* seq_off, const int* slots, const int* past, float* out, int B, int H, int D, int V,
+                       const float* gates, float* Z, float* ztmp, long tokens, int dtype, cudaStream_t s) {
   if (B == 0) return 0;
-  if (D > 256 || (!decay && !z) || (z && !zb) || (lower && !z)) return -1;
+  if (D > 256 || (!decay && !z && !gates) || (z && !zb) || (lower && !z) || (gates && (!Z || !ztmp || z || decay))) return -1;
   int dpt = D <= 64 ? 4 : 8;                    // rows per lane: 16 lanes per column group at D = 64 and at D = 128
   // few (sequence, head) pairs: the smaller tile doubles the threads per pair, which hides more of the serial walk's latency
   if (dpt == 8 && D <= 128 && (long)B * H * ((V + 127) / 128) < 100) dpt = 4;
@@ -623,19 +780,68 @@ int lbl_decay_scan(const void* q, long ldq, const void* k, long ldk, const void*
   int CT = SCAN_CT;                             // tokens per staged group: one (token, lane chunk) and one (token, column group) per thread
   while (CT > 1 && (CT * R > threads || CT * groups > threads)) CT >>= 1;
   const int Dp = R * (dpt == 8 ? 12 : 4);
-  const size_t smem = 2 * sizeof(float) * (size_t)CT * ((size_t)Dp * (z ? 3 : 2) + VT);
+  const size_t smem = 2 * sizeof(float) * (size_t)CT * ((size_t)Dp * (z ? 3 : 2) + VT + (gates ? 4 : 0));
   const dim3 grid((unsigned)(B * H), (unsigned)((V + VT - 1) / VT));
   const int esz = dtype ? 2 : 4;
   const int vec = (D % 8 == 0 && V % 8 == 0 && (ldq * esz) % 16 == 0 && (ldk * esz) % 16 == 0 && (ldv * esz) % 16 == 0 &&
                    ((uintptr_t)q & 15) == 0 && ((uintptr_t)k & 15) == 0 && ((uintptr_t)v & 15) == 0 &&
                    (!z || (ldz % 4 == 0 && ((uintptr_t)z & 15) == 0 && ((uintptr_t)zb & 15) == 0)) && ((uintptr_t)lower & 15) == 0) ? 1 : 0;
-#define DS(TT, P) { \
-    if (smem > 48 * 1024) cudaFuncSetAttribute(decay_scan_kernel<TT, P>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-    decay_scan_kernel<TT, P><<<grid, threads, smem, s>>>((const TT*)q, ldq, (const TT*)k, ldk, (const TT*)v, ldv, decay, z, ldz, zb, lower, \
-        inv_tau, q_scale, k_scale, act, S, seq_off, slots, past, out, H, D, V, R, VT, CT, vec); }
+#define DS2(TT, P, M) { \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(decay_scan_kernel<TT, P, M>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    decay_scan_kernel<TT, P, M><<<grid, threads, smem, s>>>((const TT*)q, ldq, (const TT*)k, ldk, (const TT*)v, ldv, decay, z, ldz, zb, lower, \
+        inv_tau, q_scale, k_scale, act, S, seq_off, slots, past, out, H, D, V, R, VT, CT, vec, gates, Z, ztmp, tokens); }
+#define DS(TT, P) { if (gates) DS2(TT, P, true) else DS2(TT, P, false) }
   if (dtype == 0) { if (dpt == 4) DS(float, 4) else DS(float, 8) }
   else { if (dpt == 4) DS(bf16, 4) else DS(bf16, 8) }
 #undef DS
+#undef DS2
+  if (gates && grid.y > 1) memory_keysum_kernel<<<(unsigned)(B * H), 128, 0, s>>>(ztmp, Z, slots, H, D);
+  LAUNCH_END();
+}
+
+int lbl_decay_scan(const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, const float* decay, const float* z,
+                   long ldz, const float* zb, const float* lower, float inv_tau, float q_scale, float k_scale, int act, float* S,
+                   const int* seq_off, const int* slots, const int* past, float* out, int B, int H, int D, int V, int dtype,
+                   cudaStream_t s) {
+  return launch_scan(q, ldq, k, ldk, v, ldv, decay, z, ldz, zb, lower, inv_tau, q_scale, k_scale, act, S, seq_off, slots, past, out, B, H, D, V,
+                     nullptr, nullptr, nullptr, 0, dtype, s);
+}
+
+int lbl_memory_gates(const float* z, long ldz, int foff, const float* zb, float cap, float* mx, const int* seq_off, const int* slots,
+                     const int* past, float* gates, long tokens, int B, int H, cudaStream_t s) {
+  if (B == 0 || tokens == 0) return 0;
+  if (!(cap > 0.f)) return -1;
+  memory_gates_kernel<<<(unsigned)((B * H + 3) / 4), 128, 0, s>>>(z, ldz, foff, zb, cap, mx, seq_off, slots, past, gates, tokens, B, H);
+  LAUNCH_END();
+}
+
+int lbl_memory_scan(const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, const float* gates, float q_scale, float* S,
+                    float* Z, float* ztmp, const int* seq_off, const int* slots, const int* past, float* out, long tokens, int B, int H, int D, int V,
+                    int dtype, cudaStream_t s) {
+  return launch_scan(q, ldq, k, ldk, v, ldv, nullptr, nullptr, 0, nullptr, nullptr, 1.f, q_scale, 1.f, 0, S, seq_off, slots, past, out, B, H, D, V,
+                     gates, Z, ztmp, tokens, dtype, s);
+}
+
+int lbl_memory_step(const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, const float* z, long ldz, int foff,
+                    const float* zb, float cap, float q_scale, float* S, float* Z, float* mx, const int* slots, const int* past, const void* w,
+                    const void* gate, long ldg, float eps, float out_scale, void* y, long ldy, int B, int H, int D, int V, int dtype,
+                    cudaStream_t s) {
+  if (B == 0) return 0;
+  if (!(cap > 0.f)) return -1;
+  const int nv = (V % 4 == 0 && ((uintptr_t)S & 15) == 0) ? 4 : 1, VG = (V + nv - 1) / nv;
+  int threads = 512;
+  while (threads > 64 && threads / 2 >= VG * ((D + 3) / 4)) threads /= 2;
+  int RG = threads / VG;                          // row groups that share a column group
+  if (RG < 1) RG = 1;
+  if (RG > D) RG = D;
+  const size_t smem = (2 * (size_t)D + (size_t)RG * V) * sizeof(float);
+  if (smem > 160 * 1024) return -1;
+#define MS(TT, N) { \
+    if (smem > 48 * 1024) cudaFuncSetAttribute(memory_step_kernel<TT, N>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    memory_step_kernel<TT, N><<<(unsigned)(B * H), threads, smem, s>>>((const TT*)q, ldq, (const TT*)k, ldk, (const TT*)v, ldv, z, ldz, foff, zb, cap, \
+        q_scale, S, Z, mx, slots, past, (const TT*)w, (const TT*)gate, ldg, eps, out_scale, (TT*)y, ldy, H, D, V, RG); }
+  if (dtype) { if (nv == 4) MS(bf16, 4) else MS(bf16, 1) } else { if (nv == 4) MS(float, 4) else MS(float, 1) }
+#undef MS
   LAUNCH_END();
 }
 
@@ -647,8 +853,8 @@ int lbl_gated_norm(const float* o, const void* gate, long ldg, const void* w, fl
                    ((uintptr_t)y & 15) == 0 && ((uintptr_t)w & 15) == 0) ? 1 : 0;
   if (per_head) {
     const unsigned grid = (unsigned)((rows * H * 32 + 255) / 256);
-    if (dtype) gated_norm_head_kernel<bf16><<<grid, 256, 0, s>>>(o, (const bf16*)gate, ldg, (const bf16*)w, eps, act, out_scale, (bf16*)y, ldy, rows, H, V, vec);
-    else gated_norm_head_kernel<float><<<grid, 256, 0, s>>>(o, (const float*)gate, ldg, (const float*)w, eps, act, out_scale, (float*)y, ldy, rows, H, V, vec);
+    if (dtype) gated_norm_head_kernel<bf16><<<grid, 256, 0, s>>>(o, (const bf16*)gate, ldg, (const bf16*)w, eps, act, out_scale, (bf16*)y, ldy, rows, H, V, per_head == 2, vec);
+    else gated_norm_head_kernel<float><<<grid, 256, 0, s>>>(o, (const float*)gate, ldg, (const float*)w, eps, act, out_scale, (float*)y, ldy, rows, H, V, per_head == 2, vec);
   } else {
     const int n = H * V, threads = n >= 1024 ? 256 : 128;
     if (dtype) gated_norm_row_kernel<bf16><<<(unsigned)rows, threads, 0, s>>>(o, (const bf16*)gate, ldg, (const bf16*)w, eps, act, out_scale, (bf16*)y, ldy, n, vec);

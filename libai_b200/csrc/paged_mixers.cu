@@ -164,6 +164,140 @@ __global__ void postnorm_residual_kernel(const float* xin, float* xout, const Ty
 }
 
 // ------------------------------------------------------------------------------------------------------------------
+// One sublayer boundary of a block with norms before and after its sublayers, on the fp32 residual x [rows, n] (in place):
+//   closing  (y given):   x <- x + mult * v / sqrt(mean(v^2) + eps) * (1 + pw), where v = y, or — two sublayers side by side, y2 given —
+//                         v = bscale * (y / rms(y) * bw1 + y2 / rms(y2) * bw2)
+//   entering (add given): x <- x + add                      (one row for all)
+//   opening  (h given):   h = x / sqrt(mean(x^2) + eps) * (1 + nw)
+// One block per row; the vector form keeps the row in registers (ITEMS quadruples per thread), the general one in shared memory.
+// ------------------------------------------------------------------------------------------------------------------
+__device__ __forceinline__ float sq4(float4 a) { return a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w; }
+// two sums over the block at once
+__device__ __forceinline__ float2 block_sum2(float a, float b, float* red) {
+  a = warp_sum(a); b = warp_sum(b);
+  const int w = threadIdx.x >> 5, nw = (blockDim.x + 31) >> 5;
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) { red[w] = a; red[32 + w] = b; }
+  __syncthreads();
+  float2 t = make_float2(0.f, 0.f);
+  for (int i = 0; i < nw; ++i) { t.x += red[i]; t.y += red[32 + i]; }
+  return t;
+}
+
+template <typename T, int ITEMS>
+__global__ void sandwich_residual_vec_kernel(float* __restrict__ x, const float* __restrict__ y, long ldy, const float* __restrict__ y2, long ldy2,
+                                             const T* __restrict__ bw1, const T* __restrict__ bw2, float bscale, const T* __restrict__ pw,
+                                             float mult, const T* __restrict__ add, const T* __restrict__ nw, float eps, T* __restrict__ h,
+                                             long ldh, int n) {
+  __shared__ float red[64];
+  const long row = blockIdx.x;
+  float4 xv[ITEMS], v[ITEMS];
+  float sa = 0.f, sb = 0.f;
+  float4 v2[ITEMS];
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int i = (threadIdx.x + it * blockDim.x) * 4;
+    xv[it] = v[it] = v2[it] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < n) {
+      xv[it] = ld4f(x + row * n + i);
+      if (y) { v[it] = ld4f(y + row * ldy + i); sa += sq4(v[it]); }
+      if (y2) { v2[it] = ld4f(y2 + row * ldy2 + i); sb += sq4(v2[it]); }
+    }
+  }
+  if (y) {
+    float2 t = block_sum2(sa, sb, red);
+    if (y2) {
+      const float r1 = bscale / sqrtf(t.x / (float)n + eps), r2 = bscale / sqrtf(t.y / (float)n + eps);
+      sa = 0.f;
+#pragma unroll
+      for (int it = 0; it < ITEMS; ++it) {
+        const int i = (threadIdx.x + it * blockDim.x) * 4;
+        if (i < n) {
+          const float4 a = ld4f(bw1 + i), b = ld4f(bw2 + i);
+          v[it] = make_float4(v[it].x * r1 * a.x + v2[it].x * r2 * b.x, v[it].y * r1 * a.y + v2[it].y * r2 * b.y,
+                              v[it].z * r1 * a.z + v2[it].z * r2 * b.z, v[it].w * r1 * a.w + v2[it].w * r2 * b.w);
+          sa += sq4(v[it]);
+        }
+      }
+      t.x = block_sum(sa, red);
+    }
+    const float r = mult / sqrtf(t.x / (float)n + eps);
+#pragma unroll
+    for (int it = 0; it < ITEMS; ++it) {
+      const int i = (threadIdx.x + it * blockDim.x) * 4;
+      if (i < n) {
+        const float4 w = ld4f(pw + i);
+        xv[it].x += v[it].x * r * (1.f + w.x); xv[it].y += v[it].y * r * (1.f + w.y);
+        xv[it].z += v[it].z * r * (1.f + w.z); xv[it].w += v[it].w * r * (1.f + w.w);
+      }
+    }
+  }
+  sa = 0.f;
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int i = (threadIdx.x + it * blockDim.x) * 4;
+    if (i < n) {
+      if (add) { const float4 a = ld4f(add + i); xv[it].x += a.x; xv[it].y += a.y; xv[it].z += a.z; xv[it].w += a.w; }
+      if (y || add) st4f(x + row * n + i, xv[it]);
+      sa += sq4(xv[it]);
+    }
+  }
+  if (!h) return;
+  const float r = 1.f / sqrtf(block_sum(sa, red) / (float)n + eps);
+#pragma unroll
+  for (int it = 0; it < ITEMS; ++it) {
+    const int i = (threadIdx.x + it * blockDim.x) * 4;
+    if (i < n) {
+      const float4 w = ld4f(nw + i);
+      st4f(h + row * ldh + i, make_float4(xv[it].x * r * (1.f + w.x), xv[it].y * r * (1.f + w.y), xv[it].z * r * (1.f + w.z), xv[it].w * r * (1.f + w.w)));
+    }
+  }
+}
+
+template <typename T>
+__global__ void sandwich_residual_kernel(float* __restrict__ x, const float* __restrict__ y, long ldy, const float* __restrict__ y2, long ldy2,
+                                         const T* __restrict__ bw1, const T* __restrict__ bw2, float bscale, const T* __restrict__ pw, float mult,
+                                         const T* __restrict__ add, const T* __restrict__ nw, float eps, T* __restrict__ h, long ldh, int n) {
+  extern __shared__ float sm[];                  // the sublayers' combined output, then the new residual (a thread rereads what it wrote)
+  __shared__ float red[64];
+  const long row = blockIdx.x;
+  float* xr = x + row * n;
+  float r = 0.f;
+  if (y) {
+    const float* yr = y + row * ldy;
+    const float* zr = y2 ? y2 + row * ldy2 : nullptr;
+    float sa = 0.f, sb = 0.f;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) { sa += yr[i] * yr[i]; if (zr) sb += zr[i] * zr[i]; }
+    float2 t = block_sum2(sa, sb, red);
+    if (zr) {
+      const float r1 = bscale / sqrtf(t.x / (float)n + eps), r2 = bscale / sqrtf(t.y / (float)n + eps);
+      sa = 0.f;
+      for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const float v = yr[i] * r1 * ldf(bw1 + i) + zr[i] * r2 * ldf(bw2 + i);
+        sm[i] = v;
+        sa += v * v;
+      }
+      t.x = block_sum(sa, red);
+    } else {
+      for (int i = threadIdx.x; i < n; i += blockDim.x) sm[i] = yr[i];
+    }
+    r = mult / sqrtf(t.x / (float)n + eps);
+  }
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    float v = xr[i];
+    if (y) v += sm[i] * r * (1.f + ldf(pw + i));
+    if (add) v += ldf(add + i);
+    if (y || add) xr[i] = v;
+    sm[i] = v;
+    ss += v * v;
+  }
+  if (!h) return;
+  const float rn = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+  for (int i = threadIdx.x; i < n; i += blockDim.x) stf(h + row * ldh + i, sm[i] * rn * (1.f + ldf(nw + i)));
+}
+
+// ------------------------------------------------------------------------------------------------------------------
 // Query / key / value preparation.  One warp per (token, head unit): the H query heads, then the G key heads, then the
 // G value heads.  u = the projections (three column slices with one row stride); y_t = sum_j w[c, j] u_(t - taps + 1 + j)
 // with zeros before the sequence's start, earlier steps' rows taken from `tail` [slots, taps-1, C] (row r = position
@@ -821,6 +955,35 @@ int lbp_postnorm_residual(const float* xin, float* xout, const void* y1, long ld
   if (dtype) { if (y1dtype) PN(bf16, bf16) else PN(bf16, float) }
   else { if (y1dtype) return -1; PN(float, float) }
 #undef PN
+  LAUNCH_END();
+}
+
+int lbp_sandwich_residual(float* x, const float* y, long ldy, const float* y2, long ldy2, const void* bw1, const void* bw2, float bscale,
+                          const void* pw, float mult, const void* add, const void* nw, float eps, void* h, long ldh, long rows, int n,
+                          int dtype, cudaStream_t s) {
+  if (rows == 0) return 0;
+  const size_t smem = (size_t)n * sizeof(float);
+  if (smem > 160 * 1024) return -1;
+  const int esz = dtype ? 2 : 4;
+  auto al = [&](const void* p, int a) { return ((uintptr_t)p % a) == 0; };
+  const bool vec = n % 4 == 0 && al(x, 16) && al(y, 16) && al(y2, 16) && ldy % 4 == 0 && ldy2 % 4 == 0 && ldh % 4 == 0 && al(bw1, 4 * esz) &&
+                   al(bw2, 4 * esz) && al(pw, 4 * esz) && al(add, 4 * esz) && al(nw, 4 * esz) && al(h, 4 * esz);
+#define SRA(TT) x, y, ldy, y2, ldy2, (const TT*)bw1, (const TT*)bw2, bscale, (const TT*)pw, mult, (const TT*)add, (const TT*)nw, eps, (TT*)h, ldh, n
+  if (vec && n / 4 <= 2048) {
+    const int quads = n / 4, items = quads <= 256 ? 1 : 2;
+    const int threads = (((quads + items - 1) / items + 31) / 32) * 32;
+#define SR(TT) { if (items == 1) sandwich_residual_vec_kernel<TT, 1><<<(unsigned)rows, threads, 0, s>>>(SRA(TT)); \
+                 else sandwich_residual_vec_kernel<TT, 2><<<(unsigned)rows, threads, 0, s>>>(SRA(TT)); }
+    if (dtype) SR(bf16) else SR(float)
+#undef SR
+    LAUNCH_END();
+  }
+  const int threads = n >= 2048 ? 256 : 128;
+#define SR(TT) { if (smem > 48 * 1024) cudaFuncSetAttribute(sandwich_residual_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+                 sandwich_residual_kernel<TT><<<(unsigned)rows, threads, smem, s>>>(SRA(TT)); }
+  if (dtype) SR(bf16) else SR(float)
+#undef SR
+#undef SRA
   LAUNCH_END();
 }
 

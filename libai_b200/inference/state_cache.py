@@ -8,7 +8,9 @@ A model registers one entry per layer run (a layer that is run several times in 
   of positions, ``[slots, ring_len, C]`` (position ``p`` at ``p % ring_len``), and the rows of the first ``first_len``
   positions, ``[slots, first_len, C]``, which a mask that keeps the first tokens goes on reading after they left the ring;
 * ``"recurrent"`` — the matrix state of a delta-rule or linear-attention layer, ``[slots, H, D, V]`` in fp32, and the last
-  ``taps - 1`` inputs of its short convolutions, ``[slots, taps - 1, C]`` (empty for a layer without convolutions);
+  ``taps - 1`` inputs of its short convolutions, ``[slots, taps - 1, C]`` (empty for a layer without convolutions); a layer with
+  exponential gates (``peaks=True``) also keeps the weighted sum of its keys, ``keys`` ``[slots, H, D]``, and the running maximum of
+  its log gates, ``peak`` ``[slots, H]``, both fp32;
 * ``"token"`` — the last token of the sequence, ``[slots]`` int32 (an embedding that looks at the previous token);
 * ``"paged"`` — the key/value rows (or latent rows) of an attention layer that sees the whole past: a pool ``[pages, page_size, C]`` in the compute
   dtype, shared by all sequences, and the last ``taps - 1`` inputs of the layer's short convolutions,
@@ -48,7 +50,7 @@ class SequenceStateCache:
     # ------------------------------------------------------------------ layout
     def register(self, kind: str, **shape) -> int:
         """Add one entry; returns its handle.  ``latent``: ``ring_len, channels``; ``kv``: ``ring_len, first_len, channels``;
-        ``recurrent``: ``heads, dim, vdim, taps, conv_channels``; ``token``: nothing; ``paged``: ``channels, taps,
+        ``recurrent``: ``heads, dim, vdim, taps, conv_channels`` (and ``peaks``); ``token``: nothing; ``paged``: ``channels, taps,
         conv_channels``."""
         assert kind in ("latent", "kv", "recurrent", "token", "paged"), kind
         self._paged = self._paged or kind == "paged"
@@ -67,7 +69,12 @@ class SequenceStateCache:
         if spec["kind"] == "paged":
             return {"pool": torch.zeros(self.num_pages, self.page_size, spec["channels"], dtype=self.dtype, device=self.device),
                     "tail": torch.zeros(n, max(spec["taps"] - 1, 0), spec["conv_channels"], dtype=self.dtype, device=self.device)}
+        extra = {}
+        if spec.get("peaks"):
+            extra = {"keys": torch.zeros(n, spec["heads"], spec["dim"], dtype=torch.float32, device=self.device),
+                     "peak": torch.zeros(n, spec["heads"], dtype=torch.float32, device=self.device)}
         return {
+            **extra,
             "S": torch.zeros(n, spec["heads"], spec["dim"], spec["vdim"], dtype=torch.float32, device=self.device),
             "tail": torch.zeros(n, max(spec["taps"] - 1, 0), spec["conv_channels"], dtype=self.dtype, device=self.device),
         }

@@ -20,6 +20,7 @@ from .hyper_connections import HyperConnection
 from .latent_attention import LatentAttention, PagedLatentAttention
 from .layer_norm import DynamicTanh
 from .linear_attention import DecayLinearAttention
+from .matrix_memory import MatrixMemory
 from .moe import FeedForward, GatedFeedForward, MoEFeedForward
 from .paged_attention import PagedAttention
 from .ring_attention import RingAttention

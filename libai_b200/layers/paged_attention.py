@@ -11,7 +11,12 @@ Options, all constructor arguments:
   :func:`libai_b200.ops.kv_functional.rotary_frequencies`;
 * ``talk`` — the heads' scaled scores are mixed by a learned ``[H, H]`` matrix before the mask and the softmax
   (talking-heads attention: Shazeer et al., "Talking-Heads Attention", 2020; only the mix before the softmax);
-* ``sink`` — a learned number per head whose exponential joins the softmax denominator without a key or a value.
+* ``sink`` — a learned number per head whose exponential joins the softmax denominator without a key or a value;
+* ``bias`` — the projections have biases; ``q_temp = (coef, every)`` — the query at position p is multiplied by
+  ``1 + coef · ln(⌊(p + 1) / every⌋ + 1)`` (it rides in the score scale).
+
+A layer without convolution, head norms, rotation, mix and sink (*plain*) needs no preparation: keys and values are stored as projected and
+the masked attention kernels of :mod:`libai_b200.ops.kv_functional` run on the rows (prompts) or the pages (single-token steps).
 
 State per sequence (:class:`libai_b200.inference.state_cache.SequenceStateCache`, kind ``paged``): the rows ``[keys | values]`` of
 all its positions in pages, and the last ``conv − 1`` projections.  A step prepares its rows (one kernel: convolution, norms,
@@ -43,18 +48,23 @@ def _identity_(t, generator=None):
 
 class PagedAttention(nn.Module):
     def __init__(self, width, heads, kv_heads, dim, vdim, *, scale=None, conv=1, qk_norm=True, v_norm=False, rot_dims=0, rot_base=10000.0,
-                 rot_scaling=None, talk=False, sink=False, eps=1e-6, init_method=xavier_normal_, layer_idx=0):
+                 rot_scaling=None, talk=False, sink=False, bias=False, q_temp=None, eps=1e-6, init_method=xavier_normal_, layer_idx=0):
         super().__init__()
         assert heads % kv_heads == 0 and rot_dims % 2 == 0 and rot_dims <= dim and conv >= 1
         self.width, self.heads, self.kv_heads, self.dim, self.vdim = width, heads, kv_heads, dim, vdim
         self.scale, self.eps, self.taps, self.layer_idx = float(scale if scale is not None else dim ** -0.5), eps, int(conv), layer_idx
         self.qk_norm, self.v_norm, self.rot_dims = bool(qk_norm), bool(v_norm), int(rot_dims)
-        assert self.qk_norm and self.v_norm, "the preparation kernel is built with query/key norms and unit-RMS values"
+        self.plain = not (qk_norm or v_norm or rot_dims or talk or sink) and self.taps == 1
+        assert self.plain or (self.qk_norm and self.v_norm), "the preparation kernel is built with query/key norms and unit-RMS values"
+        assert self.plain or not (bias or q_temp), "biases and query temperatures are built into the plain form"
+        self.q_temp = (float(q_temp[0]), float(q_temp[1])) if q_temp else None
         mk = lambda shape, init=init_method: create_parameter(shape, init, layer_idx=layer_idx)
         self.q, self.k, self.v = mk((heads * dim, width)), mk((kv_heads * dim, width)), mk((kv_heads * vdim, width))
         self.o = mk((width, heads * vdim))
-        self.q_conv, self.k_conv, self.v_conv = (mk((n, self.taps), _last_tap_) for n in (heads * dim, kv_heads * dim, kv_heads * vdim))
-        self.q_norm, self.k_norm = mk((dim,), ones_), mk((dim,), ones_)
+        sizes = (heads * dim, kv_heads * dim, kv_heads * vdim)
+        self.q_conv, self.k_conv, self.v_conv = (None if self.plain else mk((n, self.taps), _last_tap_) for n in sizes)
+        self.q_norm, self.k_norm = (None if self.plain else mk((dim,), ones_) for _ in range(2))
+        self.q_b, self.k_b, self.v_b = (mk((n,), zeros_) if bias else None for n in sizes)
         self.talk = mk((heads, heads), _identity_) if talk else None
         self.sink = mk((heads,), zeros_) if sink else None
         freq, mscale = KF.rotary_frequencies(self.rot_dims, rot_base, rot_scaling) if rot_dims else (torch.zeros(0), 1.0)
@@ -67,10 +77,13 @@ class PagedAttention(nn.Module):
 
     def state_spec(self):
         H, G, D, V = self.heads, self.kv_heads, self.dim, self.vdim
-        return "paged", dict(channels=G * (D + V), taps=self.taps, conv_channels=H * D + G * D + G * V)
+        return "paged", dict(channels=G * (D + V), taps=self.taps, conv_channels=0 if self.plain else H * D + G * D + G * V)
 
     def input_weights(self):
         return [("q", self.q), ("k", self.k), ("v", self.v)]
+
+    def input_biases(self):
+        return {} if self.q_b is None else {"q": self.q_b, "k": self.k_b, "v": self.v_b}
 
     def output_weight(self):
         return self.o
@@ -92,6 +105,13 @@ class PagedAttention(nn.Module):
         H, G, D, V = self.heads, self.kv_heads, self.dim, self.vdim
         if self.rot_freq.device != parts["q"].device:
             self.rot_freq = self.rot_freq.to(parts["q"].device)
+        if self.plain:
+            q, k, v, pool, table = parts["q"], parts["k"], parts["v"], bufs["pool"], bufs["table"]
+            KF.heads_prepare(q, k, v, None, None, self.rot_freq, self.eps, rb, H, G, D, V, pool=pool, table=table)
+            if rb.single:
+                return KF.page_attention(q, pool, table, None, rb, y, H, G, D, V, self.scale, out_scale=out_scale, temp=self.q_temp)
+            kmat, vmat, ext = PF.page_rows(pool, table, rb, k, v)
+            return KF.masked_attention(q, kmat, vmat, ext, None, rb, y, H, G, D, V, 0, 0, 0, self.scale, out_scale=out_scale, temp=self.q_temp)
         q = PF.conv_qkv_prepare(parts["q"], parts["k"], parts["v"], self.q_conv, self.k_conv, self.v_conv, bufs["tail"], self.q_norm,
                                 self.k_norm, self.rot_freq, self.eps, rb, bufs["pool"], bufs["table"], H, G, D, V)
         return PF.talk_attention(q, bufs["pool"], bufs["table"], rb, y, H, G, D, V, self.scale, talk=self._fp32("talk"),
@@ -99,7 +119,8 @@ class PagedAttention(nn.Module):
 
     def forward(self, h, rb, bufs, shared=None):
         """Unfused form: ``h`` ``[tokens, width]`` packed rows → ``[tokens, width]``."""
-        proj = KF.linear(h, torch.cat([self.q, self.k, self.v], 0))
+        bias = torch.cat([self.q_b, self.k_b, self.v_b]) if self.q_b is not None else None
+        proj = KF.linear(h, torch.cat([self.q, self.k, self.v], 0), bias)
         a, b = self.heads * self.dim, (self.heads + self.kv_heads) * self.dim
         parts = {"q": proj[:, :a], "k": proj[:, a:b], "v": proj[:, b:]}
         y = torch.empty(h.shape[0], self.mix_features, dtype=h.dtype, device=h.device)

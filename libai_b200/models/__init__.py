@@ -1,6 +1,7 @@
 from .bert_model import BertForClassification, BertForPreTraining, BertModel
 from .build import build_graph, build_model
 from .bumodra_model import BumodraForCausalLM, BumodraModel
+from .fogezen_model import FogezenForCausalLM, FogezenModel
 from .nefelorn_model import NefelornForCausalLM, NefelornModel
 from .gpt_model import GPTForPreTraining, GPTModel
 from .llama_model import LlamaForCausalLM, LlamaModel
@@ -22,6 +23,6 @@ __all__ = [
     "T5Model", "T5ForPreTraining",
     "VisionTransformer", "SwinTransformer", "SwinTransformerV2", "ResMLP",
     "LlamaModel", "LlamaForCausalLM",
-    "BumodraModel", "BumodraForCausalLM", "NefelornModel", "NefelornForCausalLM",
+    "BumodraModel", "BumodraForCausalLM", "FogezenModel", "FogezenForCausalLM", "NefelornModel", "NefelornForCausalLM",
     "SalizenModel", "SalizenForCausalLM", "VoduzenModel", "VoduzenForCausalLM", "ZubaraxModel", "ZubaraxForCausalLM",
 ]

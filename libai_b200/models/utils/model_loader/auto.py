@@ -49,6 +49,13 @@ def _zubarax():
     return ZubaraxForCausalLM, ZubaraxLoader, {}
 
 
+def _fogezen():
+    from libai_b200.models import FogezenForCausalLM
+    from .fogezen_loader import FogezenLoader
+
+    return FogezenForCausalLM, FogezenLoader, {}
+
+
 def _voduzen():
     from libai_b200.models import VoduzenForCausalLM
     from .voduzen_loader import VoduzenLoader
@@ -58,6 +65,7 @@ def _voduzen():
 
 ARCHITECTURES = {
     "bumodra": _bumodra,
+    "fogezen": _fogezen,
     "nefelorn": _nefelorn,
     "salizen": _salizen,
     "voduzen": _voduzen,
@@ -67,7 +75,7 @@ ARCHITECTURES = {
 
 
 # native libraries (``libai_b200.ops.build``) that a model's generation path launches besides the GEMM library ``_C``
-NATIVE_LIBS = {"bumodra": ["_C_seq"], "nefelorn": ["_C_kv"], "salizen": ["_C_kv", "_C_lin"],
+NATIVE_LIBS = {"bumodra": ["_C_seq"], "fogezen": ["_C_kv", "_C_lin"], "nefelorn": ["_C_kv"], "salizen": ["_C_kv", "_C_lin"],
                "voduzen": ["_C_kv"], "zubarax": ["_C_kv", "_C_lin"]}
 
 

@@ -192,6 +192,47 @@ def qk_prepare(q, k, qw, kw, freq, mscale: float, rb, H: int, G: int, D: int, ep
         t.copy_(v.reshape(-1, heads * D))
 
 
+def heads_prepare(q, k, v, qn, kn, freq, eps: float, rb, H: int, G: int, D: int, V: int, *, pairs: bool = True, ring=None, pool=None,
+                  table=None):
+    """Per-head preparation and cache write in one pass.  ``q`` ``[tokens, H·D]`` and ``k`` ``[tokens, G·D]``, in place: RMS norm of every
+    head with the weights ``qn`` / ``kn`` ``[D]`` shared by the heads (``None``: no norm), then rotation of the first ``2·len(freq)``
+    channels by ``position · freq[i]``, channel ``2i`` with ``2i + 1`` (``pairs``) or ``i`` with ``i + len(freq)``.  The keys so prepared and the
+    values ``v`` ``[tokens, G·V]`` go to the row of their position in ``ring`` ``[slots, L, G·D + G·V]`` (position p at ``p % L``) or in the pages
+    of ``pool`` / ``table`` (neither: nothing is stored)."""
+    cache = ring if ring is not None else pool
+    if _native(q):
+        if cache is None and qn is None and freq.numel() == 0:
+            return
+        count_launch()
+        load_kv_ext().heads_prepare(q, k, v, qn, kn, freq, bool(pairs), float(eps), cache, table if ring is None else None, rb.tok_seq, rb.seq_off,
+                                    rb.slots, rb.past, H, G, D, V)
+        return
+    half = freq.numel()
+    if qn is not None or half:
+        pos = torch.cat([torch.arange(p, p + n) for p, n in zip(rb.past_list, rb.lens)]).to(q.device).float()
+        ang = (pos[:, None] * freq.float()[None, :])[:, None, :]
+        cos, sin = ang.cos(), ang.sin()
+        for t, w, heads in ((q, qn, H), (k, kn, G)):
+            u = t.float().view(-1, heads, D)
+            if w is not None:
+                u = u * torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+            if half:
+                a, b = (u[..., 0:2 * half:2], u[..., 1:2 * half:2]) if pairs else (u[..., :half], u[..., half:2 * half])
+                a, b = a * cos - b * sin, b * cos + a * sin
+                u = torch.cat([torch.stack([a, b], -1).flatten(-2) if pairs else torch.cat([a, b], -1), u[..., 2 * half:]], -1)
+            t.copy_(u.reshape(-1, heads * D))
+    if cache is None:
+        return
+    if ring is not None:
+        kv_write(ring, ring[:, :0], k, v, rb)
+        return
+    ps = pool.shape[1]
+    for b in range(rb.B):
+        lo, n, past = rb.offsets[b], rb.lens[b], rb.past_list[b]
+        p = torch.arange(past, past + n, device=table.device)
+        pool[table[rb.slot_list[b], p // ps].long(), p % ps] = torch.cat([k[lo:lo + n], v[lo:lo + n]], 1)
+
+
 # ----------------------------------------------------------------------------------------------------------- cache rows
 def kv_write(ring, first, knew, vnew, rb):
     """Store the step's key / value rows: position p of a sequence goes to ``ring[slot, p % L]`` and, for ``p < nfirst``, to
@@ -261,6 +302,11 @@ def _attend_rows(qrow, keys, vals, H, G, D, V, scale, softcap=0.0, sink=False):
     return torch.einsum("hj,jhv->hv", p, v)
 
 
+def query_temperature(position: int, temp):
+    """``1 + coef · ln(⌊(position + 1) / every⌋ + 1)`` for ``temp = (coef, every)``; 1 without one."""
+    return 1.0 + temp[0] * math.log(math.floor((position + 1) / temp[1]) + 1.0) if temp else 1.0
+
+
 def _gated(o, gate_row, wide: bool, out_scale: float):
     """``o`` ``[H, V]`` times ``sigmoid`` of the row's gate logits (one per head, or — ``wide`` — one per channel) and ``out_scale``."""
     if gate_row is not None:
@@ -271,29 +317,31 @@ def _gated(o, gate_row, wide: bool, out_scale: float):
 
 def masked_attention(q, kmat, vmat, ext, gate, rb, y, H: int, G: int, D: int, V: int, window: int, chunk: int, keep: int,
                      scale: float, mma: bool = True, softcap: float = 0.0, sink: bool = False, gate_wide: bool = False,
-                     out_scale: float = 1.0):
+                     out_scale: float = 1.0, temp=None):
     """Grouped-query softmax attention of every packed query over the rows of the ext matrix (``kmat`` ``[rows, G·D]``,
     ``vmat`` ``[rows, G·V]``: column slices with one row stride) that its mask admits: position j ≤ i with
     ``j ≥ ⌊i/chunk⌋·chunk`` (``chunk > 0``) or ``j > i − window or j < keep`` (``window > 0``).  Head h of the result is
     multiplied by ``sigmoid(gate[t, h])`` when a gate is given (``gate_wide``: channel c of head h by
     ``sigmoid(gate[t, h·V + c])``) and by ``out_scale``.  ``softcap`` > 0: scaled scores pass through ``cap · tanh(s / cap)``;
-    ``sink``: the softmax has one more entry of score 0 without a value.  bf16 inputs with head sizes the tensor-core kernel is
-    built for take it; ``mma=False`` keeps them on the generic kernel (fp32 inputs always are)."""
+    ``sink``: the softmax has one more entry of score 0 without a value; ``temp = (coef, every)``: the query at position p is
+    multiplied by ``1 + coef · ln(⌊(p + 1) / every⌋ + 1)``.  bf16 inputs with head sizes the tensor-core kernel is built for take it;
+    ``mma=False`` keeps them on the generic kernel (fp32 inputs always are)."""
     if _native(q):
         count_launch()
+        coef, every = temp if temp else (0.0, 0.0)
         tiles = (None, None)
         if mma and q.dtype == torch.bfloat16 and mma_eligible(q, kmat, vmat, y, D, V) and (
                 gate is None or not gate_wide or (gate.data_ptr() % 4 == 0 and gate.stride(0) % 2 == 0 and V % 2 == 0)):
             tiles = rb.query_tiles(64)
         load_kv_ext().masked_attention(q, kmat, vmat, ext.ext_off, ext.nsink, ext.cstart, gate, rb.tok_seq, rb.seq_off, rb.past,
                                        tiles[0], tiles[1], y, H, G, D, V, window, chunk, keep, float(scale), float(softcap), bool(sink),
-                                       bool(gate_wide), float(out_scale))
+                                       bool(gate_wide), float(out_scale), float(coef), float(every))
         return y
     for b in range(rb.B):
         lo, n, past, eo, ns, cs = rb.offsets[b], rb.lens[b], rb.past_list[b], ext.offsets[b], ext.nsink_list[b], ext.cstart_list[b]
         for t in range(n):
             rows = [eo + (p if p < cs else ns + p - cs) for p in _visible(past + t, window, chunk, keep)]
-            o = _attend_rows(q[lo + t], kmat[rows], vmat[rows], H, G, D, V, scale, softcap, sink)
+            o = _attend_rows(q[lo + t], kmat[rows], vmat[rows], H, G, D, V, scale * query_temperature(past + t, temp), softcap, sink)
             o = _gated(o, None if gate is None else gate[lo + t], gate_wide, out_scale)
             y[lo + t] = o.reshape(-1).to(y.dtype)
     return y
@@ -301,6 +349,11 @@ def masked_attention(q, kmat, vmat, ext, gate, rb, y, H: int, G: int, D: int, V:
 
 MMA_HEAD_SIZES = (32, 48, 64, 96, 128)       # head sizes (keys = values) the tensor-core prompt kernel is built for
 GROUPED_DECODE = True                      # single-token steps: the grouped split kernel where its sizes allow
+PAGE_DECODE_BLOCKS = 592                   # blocks a single-token step over pages is cut into (four per SM)
+
+
+def grouped_decode_ok(H: int, G: int, D: int, V: int) -> bool:
+    return GROUPED_DECODE and H // G <= 8 and V <= 128 and (H // G * D + 4 * H // G * (V + 2)) * 4 <= 48 * 1024
 
 
 def mma_eligible(q, kmat, vmat, y, D: int, V: int) -> bool:
@@ -309,29 +362,53 @@ def mma_eligible(q, kmat, vmat, y, D: int, V: int) -> bool:
 
 def ring_attention(q, ring, first, gate, rb, y, H: int, G: int, D: int, V: int, window: int, chunk: int, keep: int, scale: float,
                    splits: Optional[int] = None, softcap: float = 0.0, sink: bool = False, gate_wide: bool = False,
-                   out_scale: float = 1.0):
+                   out_scale: float = 1.0, temp=None):
     """Single-token steps: the same attention with keys and values read straight from ``ring`` / ``first`` (the step's own row
     has been written).  ``splits``: 0 = one warp per (token, head); n > 0 = the grouped kernel with the visible keys of a
-    (sequence, key head) cut into n parts; ``None`` chooses by the mask's reach.  ``softcap``, ``sink``, ``gate_wide`` and
-    ``out_scale`` as in :func:`masked_attention`."""
+    (sequence, key head) cut into n parts; ``None`` chooses by the mask's reach.  ``softcap``, ``sink``, ``gate_wide``,
+    ``out_scale`` and ``temp`` as in :func:`masked_attention`."""
     if _native(q):
+        coef, every = temp if temp else (0.0, 0.0)
         if splits is None:
             reach = (chunk if chunk > 0 else window) + keep
-            if not GROUPED_DECODE or H // G > 8 or V > 128 or (H // G * D + 4 * H // G * (V + 2)) * 4 > 48 * 1024:
+            if not grouped_decode_ok(H, G, D, V):
                 splits = 0
             else:                                               # enough blocks for the device, at least 64 positions each
                 splits = max(1, min(32, (reach + 63) // 64, -(-296 // (q.shape[0] * G))))
         count_launch(1 if splits == 0 else 2)
         load_kv_ext().ring_attention(q, ring, first, gate, rb.tok_seq, rb.seq_off, rb.slots, rb.past, y, H, G, D, V, window, chunk, keep,
-                                     float(scale), splits, float(softcap), bool(sink), bool(gate_wide), float(out_scale))
+                                     float(scale), splits, float(softcap), bool(sink), bool(gate_wide), float(out_scale), float(coef), float(every))
         return y
     L, nf, KC = ring.shape[1], first.shape[1], G * D
     for b in range(rb.B):
         slot, pi = rb.slot_list[b], rb.past_list[b]
         rows = torch.stack([first[slot, p] if p < nf else ring[slot, p % L] for p in _visible(pi, window, chunk, keep)])
-        o = _attend_rows(q[b], rows[:, :KC], rows[:, KC:], H, G, D, V, scale, softcap, sink)
+        o = _attend_rows(q[b], rows[:, :KC], rows[:, KC:], H, G, D, V, scale * query_temperature(pi, temp), softcap, sink)
         o = _gated(o, None if gate is None else gate[b], gate_wide, out_scale)
         y[b] = o.reshape(-1).to(y.dtype)
+    return y
+
+
+def page_attention(q, pool, table, gate, rb, y, H: int, G: int, D: int, V: int, scale: float, splits: Optional[int] = None, softcap: float = 0.0,
+                   sink: bool = False, gate_wide: bool = False, out_scale: float = 1.0, temp=None):
+    """Single-token steps over a paged cache (``pool`` ``[pages, page_size, G·D + G·V]``, ``table`` ``[slots, max_pages]``): every query sees
+    the whole past of its sequence (the step's own row has been written).  Options as in :func:`ring_attention`; the number of parts
+    does not depend on how long the sequences are, so that a captured step stays right as they grow."""
+    if _native(q):
+        coef, every = temp if temp else (0.0, 0.0)
+        if splits is None:
+            splits = max(1, min(32, -(-PAGE_DECODE_BLOCKS // (q.shape[0] * G)))) if grouped_decode_ok(H, G, D, V) else 0
+        count_launch(1 if splits == 0 else 2)
+        load_kv_ext().page_attention(q, pool, table, gate, rb.tok_seq, rb.seq_off, rb.slots, rb.past, y, H, G, D, V, float(scale), splits,
+                                     float(softcap), bool(sink), bool(gate_wide), float(out_scale), float(coef), float(every))
+        return y
+    KC, ps = G * D, pool.shape[1]
+    for b in range(rb.B):
+        pi = rb.past_list[b]
+        p = torch.arange(pi + 1, device=table.device)
+        rows = pool[table[rb.slot_list[b], p // ps].long(), p % ps]
+        o = _attend_rows(q[b], rows[:, :KC], rows[:, KC:], H, G, D, V, scale * query_temperature(pi, temp), softcap, sink)
+        y[b] = _gated(o, None if gate is None else gate[b], gate_wide, out_scale).reshape(-1).to(y.dtype)
     return y
 
 

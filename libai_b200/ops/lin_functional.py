@@ -117,14 +117,68 @@ def decay_scan(q, k, v, S, rb, *, decay=None, z=None, zb=None, tau: float = 1.0,
     return out
 
 
+def memory_gates(z, zb, foff: int, cap: float, H: int):
+    """Log input and log forget gates ``[tokens, H]`` from the fp32 logits: ``cap · tanh((z + b) / cap)``, the forget gate through
+    ``log sigmoid``; the input gates' logits are the columns ``0 …``, the forget gates' ``foff …``."""
+    u = cap * torch.tanh((z + zb) / cap)
+    return u[:, :H], F.logsigmoid(u[:, foff:foff + H])
+
+
+def memory_scan(q, k, v, z, zb, foff: int, cap: float, q_scale: float, bufs, rb):
+    """The matrix memory with exponential gates over the packed rows (``q``, ``k`` ``[tokens, H·D]``, ``v`` ``[tokens, H·V]``): with the
+    log gates ``i``, ``f`` of :func:`memory_gates` and a running maximum ``m`` (0 at the start of a sequence),
+    ``m' = max(f + m, i)``, ``S ← e^(f+m−m') S + e^(i−m') k vᵀ``, ``z ← …`` likewise with ``k`` alone, and the read-out is
+    ``Sᵀq / (max(|z·q|, e^(−m')) + 1e-6)``.  ``bufs``: ``S`` ``[slots, H, D, V]``, ``keys`` (the sums ``z``) ``[slots, H, D]`` and ``peak`` (``m``)
+    ``[slots, H]``, all fp32; they are read unless ``past == 0`` and left at the state after the last row.  Returns fp32 ``[tokens, H·V]``."""
+    S, Z, mx = bufs["S"], bufs["keys"], bufs["peak"]
+    H, D, V = S.shape[1:]
+    out = torch.empty(q.shape[0], H * V, dtype=torch.float32, device=q.device)
+    if _native(q):
+        count_launch(2)
+        load_lin_ext().memory_scan(q, k, v, z, zb, int(foff), float(cap), float(q_scale), S, Z, mx, rb.seq_off, rb.slots, rb.past, out)
+        return out
+    li, lf = memory_gates(z, zb, foff, cap, H)
+    for b in range(rb.B):
+        lo, n, slot = rb.offsets[b], rb.lens[b], rb.slot_list[b]
+        fresh = rb.past_list[b] == 0
+        st, zs, m = (torch.zeros_like(t[slot]) if fresh else t[slot].clone() for t in (S, Z, mx))
+        qq, kk, vv = (q[lo:lo + n].float() * q_scale).view(n, H, D), k[lo:lo + n].float().view(n, H, D), v[lo:lo + n].float().view(n, H, V)
+        for t in range(n):
+            i, f = li[lo + t], lf[lo + t]
+            new = torch.maximum(f + m, i)
+            keep, put = torch.exp(f + m - new), torch.exp(i - new)
+            m = new
+            kt = put[:, None] * kk[t]
+            st = keep[:, None, None] * st + kt[:, :, None] * vv[t][:, None, :]
+            zs = keep[:, None] * zs + kt
+            div = torch.maximum((zs * qq[t]).sum(-1).abs(), torch.exp(-m)) + 1e-6
+            out[lo + t] = (torch.einsum("hdv,hd->hv", st, qq[t]) / div[:, None]).reshape(-1)
+        S[slot], Z[slot], mx[slot] = st, zs, m
+    return out
+
+
+def memory_step(q, k, v, z, zb, foff: int, cap: float, q_scale: float, bufs, rb, w, gate, eps: float, y, out_scale: float = 1.0):
+    """Single-token steps in one kernel: :func:`memory_scan`, then every head divided by its root mean square, times ``w`` ``[H·V]``,
+    ``sigmoid(gate)`` and ``out_scale``, into ``y`` ``[tokens, H·V]``."""
+    S = bufs["S"]
+    if _native(q):
+        count_launch()
+        load_lin_ext().memory_step(q, k, v, z, zb, int(foff), float(cap), float(q_scale), S, bufs["keys"], bufs["peak"], rb.slots, rb.past, w, gate,
+                                   float(eps), float(out_scale), y)
+        return y
+    o = memory_scan(q, k, v, z, zb, foff, cap, q_scale, bufs, rb)
+    return gated_norm(o, gate, w, eps, GATE_NONE if gate is None else GATE_SIGMOID, y, S.shape[1], S.shape[3], per_head=True, out_scale=out_scale)
+
+
 def gated_norm(o, gate, w, eps: float, act: int, y, H: int, V: int, *, per_head: bool, out_scale: float = 1.0):
     """``y = o / sqrt(mean(o²) + eps) · w · act(gate) · out_scale`` for the fp32 read-outs ``o`` ``[rows, H·V]``; the mean runs
-    over the ``V`` channels of every head (``per_head``; ``w`` ``[V]`` shared by the heads) or over the whole row (``w``
+    over the ``V`` channels of every head (``per_head``; ``w`` ``[V]`` shared by the heads, or ``[H·V]``) or over the whole row (``w``
     ``[H·V]``); ``w = None`` leaves the weight out; ``act``: ``GATE_SILU``, ``GATE_SIGMOID`` or ``GATE_NONE`` (no gate: ``gate`` may be
     ``None``)."""
     if _native(o):
         count_launch()
-        load_lin_ext().gated_norm(o, gate, w, float(eps), int(act), float(out_scale), y, H, V, bool(per_head))
+        wide = per_head and w is not None and w.numel() == H * V and H > 1
+        load_lin_ext().gated_norm(o, gate, w, float(eps), int(act), float(out_scale), y, H, V, bool(per_head), wide)
         return y
     of = o.view(-1, H, V) if per_head else o.view(-1, 1, H * V)
     v = of * torch.rsqrt(of.pow(2).mean(-1, keepdim=True) + eps) * out_scale
@@ -132,6 +186,6 @@ def gated_norm(o, gate, w, eps: float, act: int, y, H: int, V: int, *, per_head:
         g = gate.float().reshape(of.shape)
         v = v * (F.silu(g) if act == GATE_SILU else torch.sigmoid(g))
     if w is not None:
-        v = v * w.float()
+        v = v * (w.float().view(H, V) if per_head and w.numel() == H * V else w.float())
     y.copy_(v.reshape(-1, H * V))
     return y

@@ -61,6 +61,29 @@ def outnorm_residual(x, w, eps: float, *, y=None, y2=None, pos=None, cw=None, ga
     return postnorm_residual(x, w, eps, alpha=0.0, y=y, y2=y2, pos=pos, cw=cw, h=h, gate=gate, keep=keep, outer=True)
 
 
+def sandwich_residual(x, eps: float, *, y=None, post=None, mult: float = 1.0, y2=None, branch=None, branch_scale: float = 0.5, add=None,
+                      nxt=None, h=None):
+    """One sublayer boundary of blocks with RMS norms before and after their sublayers, on the fp32 residual ``x`` ``[rows, width]`` (in
+    place), every step optional: closing — ``x += mult · norm(v; 1 + post)`` with ``v = y`` (fp32), or, with a second output ``y2`` and
+    ``branch = (w, w2)``, ``v = branch_scale · (norm(y; w) + norm(y2; w2))``; entering — ``x += add`` (one row for all); opening —
+    ``h = norm(x; 1 + nxt)`` in the compute dtype.  ``norm(t; w) = t / sqrt(mean(t²) + eps) · w``."""
+    if _native(x):
+        count_launch()
+        w1, w2 = branch if y2 is not None else (None, None)
+        load_kv_ext().sandwich_residual(x, y, y2, w1, w2, float(branch_scale), post if y is not None else None, float(mult), add,
+                                        nxt if h is not None else None, float(eps), h)
+        return x
+    unit = lambda t: t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps)
+    if y is not None:
+        v = y if y2 is None else branch_scale * (unit(y) * branch[0].float() + unit(y2) * branch[1].float())
+        x.add_(mult * unit(v) * (1.0 + post.float()))
+    if add is not None:
+        x.add_(add.float())
+    if h is not None:
+        h.copy_(unit(x) * (1.0 + nxt.float()))
+    return x
+
+
 # ------------------------------------------------------------------------------------------------- query / key / value rows
 def _page_rows(table, slot: int, lo: int, hi: int, page_size: int):
     """(page, row) of the positions ``lo … hi - 1`` of the sequence in ``slot``."""
@@ -113,6 +136,23 @@ def conv_qkv_prepare(q, k, v, wq, wk, wv, tail, qn, kn, freq, eps: float, rb, po
         page, row = _page_rows(table, slot, past, past + n, ps)
         pool[page, row] = torch.cat([turn(yk).reshape(n, G * D), yv.reshape(n, G * V)], 1).to(pool.dtype)
     return qout
+
+
+def page_rows(pool, table, rb, k, v):
+    """Keys and values of a prompt step over the whole past, as column slices of one matrix, and the step's row layout
+    (:class:`~libai_b200.inference.ragged.KvExt`): the step's own rows when every sequence starts at position 0, otherwise a gather of
+    every sequence's pages (the step's rows have been written)."""
+    ext = rb.kv_ext([(0, 0, 0)])
+    if not ext.cached:
+        return k, v, ext
+    KC = k.shape[1]
+    if _native(pool):
+        rows = torch.empty(ext.rows, pool.shape[2], dtype=pool.dtype, device=pool.device)
+        count_launch()
+        load_kv_ext().latent_pages_gather(pool, table, ext.ext_seq, ext.ext_off, rb.slots, rows)
+    else:
+        rows = torch.cat([pool[_page_rows(table, s, 0, p + n, pool.shape[1])] for s, p, n in zip(rb.slot_list, rb.past_list, rb.lens)])
+    return rows[:, :KC], rows[:, KC:], ext
 
 
 # --------------------------------------------------------------------------------------------------------------- attention

@@ -239,8 +239,8 @@ def head_gate(x, gate, y, H: int, V: int):
 
 
 # ------------------------------------------------------------------------------------------------------------ projections
-def linear(a, w):
-    """``a @ wᵀ`` for a row-major view ``a`` ``[rows, K]`` (its rows may be a column slice of a wider matrix): the tcgen05
+def linear(a, w, bias=None):
+    """``a @ wᵀ (+ bias)`` for a row-major view ``a`` ``[rows, K]`` (its rows may be a column slice of a wider matrix): the tcgen05
     GEMM reads the slice in place through its row stride; shapes it does not take, fp32 operands and CPU tensors go to the
     vendor / PyTorch product."""
     from . import load_ext, use_native
@@ -248,16 +248,16 @@ def linear(a, w):
     if (a.is_cuda and a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and use_native(a) and a.dim() == 2
             and a.stride(1) == 1 and a.stride(0) % 8 == 0 and a.shape[1] % 8 == 0 and w.is_contiguous()
             and w.shape[0] % 8 == 0 and a.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0 and a.shape[0] > 0):
-        y = _tcgen05_gemm(a, w, None, False, torch.bfloat16)
+        y = _tcgen05_gemm(a, w, None, False, torch.bfloat16, bias)
         if y is not None:
             return y
-    return F.linear(a, w)
+    return F.linear(a, w, bias)
 
 
 _GEMM_REFUSED = set()
 
 
-def _tcgen05_gemm(a, w, out, accumulate, out_dtype):
+def _tcgen05_gemm(a, w, out, accumulate, out_dtype, bias=None):
     """The framework's GEMM; a shape it refuses (the launcher returns an error code before anything runs) is remembered and
     sent to the vendor product from then on — ``None`` tells the caller to do so."""
     from . import load_ext
@@ -266,7 +266,7 @@ def _tcgen05_gemm(a, w, out, accumulate, out_dtype):
     if key in _GEMM_REFUSED:
         return None
     try:
-        y = load_ext().gemm(a, w, 0, None, out, accumulate, out_dtype)
+        y = load_ext().gemm(a, w, 0, bias, out, accumulate, out_dtype)
     except RuntimeError as e:
         if "failed with code -" not in str(e):          # a CUDA error, not a refusal by the launcher's shape checks
             raise
@@ -290,6 +290,17 @@ def fuse_rows(named, align: int = 8):
             parts.append(w.new_zeros(pad, w.shape[1]))
         at += n + pad
     return torch.cat(parts, 0).contiguous(), where
+
+
+def fuse_biases(named, where, align: int = 8):
+    """The biases ``{name: [n_i]}`` of the segments that :func:`fuse_rows` laid out (zeros where a segment has none)."""
+    total = max(lo + n + (-n) % align for lo, n in where.values())
+    some = next(iter(named.values()))
+    out = some.new_zeros(total)
+    for name, b in named.items():
+        lo, n = where[name]
+        out[lo:lo + n] = b
+    return out
 
 
 def fuse_cols(named, align: int = 8):
