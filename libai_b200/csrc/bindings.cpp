@@ -78,6 +78,10 @@ struct LbRngArgs {
 int lb_latent_prompt_tc(const void* q, long ldq, const void* kv, long ldkv, const void* rot, long ldr, const float* cs, const float* sink,
                         const int* ext_off, const int* qt_seq, const int* qt_start, int ntiles, const int* seq_off, const int* past, void* y,
                         long ldy, long tokens, long rows, int H, int D, int R, int V, float scale, int* err, cudaStream_t s);
+int lb_masked_attention_tc(const void* q, long ldq, const void* kmat, const void* vmat, long ldkv, const int* ext_off, const int* nsink, const int* cstart,
+                           const void* gate, long ldg, int gate_wide, const int* qt_seq, const int* qt_start, int ntiles,
+                           const int* seq_off, const int* past, void* y, long ldy, long tokens, long rows, int H, int G, int D, int V,
+                           int window, int chunk, float scale, float out_scale, float temp_coef, float temp_every, int* err, cudaStream_t s);
 int lb_attn_fwd(const void* q, const void* k, const void* v, void* o, float* lse, int B, int A, int S, int D,
                 const long* q_strides, const long* k_strides, const long* v_strides, int causal, float scale,
                 const int* kv_lens, const void* bias, const long* bias_strides, const float* alibi_slopes, float p_drop,
@@ -172,6 +176,47 @@ void gemm_grouped(const Tensor& a, const Tensor& w, const std::vector<int64_t>& 
   }
 }
 
+// a mapped host word that a kernel sets when one of its bounded waits ran out; `what` has its own, checked before every launch
+struct WaitWord {
+  int* host = nullptr;
+  int* device(const char* what) {
+    if (host == nullptr) {
+      TORCH_CHECK(cudaHostAlloc(reinterpret_cast<void**>(&host), sizeof(int), cudaHostAllocMapped) == cudaSuccess, what, ": mapped host word");
+      *host = 0;
+    }
+    TORCH_CHECK(*static_cast<volatile int*>(host) == 0, what, ": a wait ran out in an earlier launch; its result is invalid");
+    int* dev = nullptr;
+    TORCH_CHECK(cudaHostGetDevicePointer(reinterpret_cast<void**>(&dev), host, 0) == cudaSuccess, what, ": mapped host word");
+    return dev;
+  }
+};
+
+// Attention of ragged prompts under a position mask (csrc/masked_attention_sm100.cu): q [tokens, H*D], kmat [rows, G*D] and vmat [rows, G*V]
+// column slices with one row stride, query tiles of 128
+void masked_attention_tc(const Tensor& q, const Tensor& kmat, const Tensor& vmat, const Tensor& ext_off, const Tensor& nsink, const Tensor& cstart,
+                         const c10::optional<Tensor>& gate, bool gate_wide, const Tensor& seq_off, const Tensor& past, const Tensor& qt_seq,
+                         const Tensor& qt_start, Tensor y, int64_t H, int64_t G, int64_t D, int64_t V, int64_t window, int64_t chunk, double scale,
+                         double out_scale, double temp_coef, double temp_every) {
+  const bool gated = gate.has_value() && gate->defined();
+  for (const Tensor* t : {&q, &kmat, &vmat, (const Tensor*)&y, gated ? &*gate : &q})
+    TORCH_CHECK(t->is_cuda() && t->dim() == 2 && (t->size(1) == 1 || t->stride(1) == 1) && t->scalar_type() == at::kBFloat16, "masked_attention_tc: bf16 row-major matrices expected");
+  TORCH_CHECK(q.size(1) == H * D && kmat.size(1) == G * D && vmat.size(1) == G * V && kmat.size(0) == vmat.size(0) && kmat.stride(0) == vmat.stride(0) &&
+              y.size(0) == q.size(0) && y.size(1) == H * V && (!gated || (gate->size(0) == q.size(0) && gate->size(1) == (gate_wide ? H * V : H))),
+              "masked_attention_tc: shapes");
+  for (const Tensor* t : {&ext_off, &nsink, &cstart, &seq_off, &past, &qt_seq, &qt_start})
+    TORCH_CHECK(t->is_cuda() && t->scalar_type() == at::kInt && t->is_contiguous(), "masked_attention_tc: int32 CUDA metadata expected");
+  TORCH_CHECK(qt_seq.numel() == qt_start.numel() && ext_off.numel() == seq_off.numel() && past.numel() + 1 == seq_off.numel() && cstart.numel() == past.numel() && nsink.numel() == past.numel(),
+              "masked_attention_tc: metadata sizes");
+  static WaitWord word;
+  int* err = word.device("masked_attention_tc");
+  c10::cuda::CUDAGuard guard(q.device());
+  check(lb_masked_attention_tc(q.data_ptr(), q.stride(0), kmat.data_ptr(), vmat.data_ptr(), kmat.stride(0), ext_off.data_ptr<int>(), nsink.data_ptr<int>(), cstart.data_ptr<int>(),
+                               gated ? gate->data_ptr() : nullptr, gated ? gate->stride(0) : 0, gate_wide ? 1 : 0, qt_seq.data_ptr<int>(),
+                               qt_start.data_ptr<int>(), (int)qt_seq.numel(), seq_off.data_ptr<int>(), past.data_ptr<int>(), y.data_ptr(), y.stride(0),
+                               q.size(0), kmat.size(0), (int)H, (int)G, (int)D, (int)V, (int)window, (int)chunk, (float)scale, (float)out_scale,
+                               (float)temp_coef, (float)temp_every, err, cur_stream()), "masked_attention_tc");
+}
+
 // Causal attention of ragged prompts on expanded latents (csrc/latent_attention_sm100.cu): q [tokens, H*(D+R)] with the R part
 // unrotated, kv [rows, H*D | H*V], rot [rows, R] the shared rotated key part, cs [tokens, R/2, 2]; query tiles of 128
 void latent_prompt_tc(const Tensor& q, const Tensor& kv, const Tensor& rot, const Tensor& cs, const c10::optional<Tensor>& sink, const Tensor& ext_off,
@@ -190,14 +235,8 @@ void latent_prompt_tc(const Tensor& q, const Tensor& kv, const Tensor& rot, cons
     TORCH_CHECK(sink->is_cuda() && sink->scalar_type() == at::kFloat && sink->is_contiguous() && sink->numel() == H, "latent_prompt_tc: sink fp32 [H]");
     sp = sink->data_ptr<float>();
   }
-  static int* err = nullptr;                     // mapped host word: a kernel whose bounded wait ran out sets it
-  if (err == nullptr) {
-    TORCH_CHECK(cudaHostAlloc(reinterpret_cast<void**>(&err), sizeof(int), cudaHostAllocMapped) == cudaSuccess, "latent_prompt_tc: mapped host word");
-    *err = 0;
-  }
-  TORCH_CHECK(*static_cast<volatile int*>(err) == 0, "latent_prompt_tc: a wait ran out in an earlier launch; its result is invalid");
-  int* err_dev = nullptr;
-  TORCH_CHECK(cudaHostGetDevicePointer(reinterpret_cast<void**>(&err_dev), err, 0) == cudaSuccess, "latent_prompt_tc: mapped host word");
+  static WaitWord word;
+  int* err_dev = word.device("latent_prompt_tc");
   c10::cuda::CUDAGuard guard(q.device());
   check(lb_latent_prompt_tc(q.data_ptr(), q.stride(0), kv.data_ptr(), kv.stride(0), rot.data_ptr(), rot.stride(0), cs.data_ptr<float>(), sp,
                             ext_off.data_ptr<int>(), qt_seq.data_ptr<int>(), qt_start.data_ptr<int>(), (int)qt_seq.numel(), seq_off.data_ptr<int>(),
@@ -871,6 +910,7 @@ TORCH_LIBRARY(libai_b200, m) {
   m.def("gemm(Tensor a, Tensor b, int layout, Tensor? bias, Tensor? out, bool accumulate, ScalarType out_dtype) -> Tensor", &gemm);
   m.def("gemm_grouped(Tensor a, Tensor w, int[] counts, Tensor(a!) out) -> ()", &gemm_grouped);
   m.def("gemm_grouped_blocks(Tensor a, Tensor w, Tensor tile_group, Tensor(a!) out) -> ()", &gemm_grouped_blocks);
+  m.def("masked_attention_tc(Tensor q, Tensor kmat, Tensor vmat, Tensor ext_off, Tensor nsink, Tensor cstart, Tensor? gate, bool gate_wide, Tensor seq_off, Tensor past, Tensor qt_seq, Tensor qt_start, Tensor(a!) y, int H, int G, int D, int V, int window, int chunk, float scale, float out_scale, float temp_coef, float temp_every) -> ()", &masked_attention_tc);
   m.def("latent_prompt_tc(Tensor q, Tensor kv, Tensor rot, Tensor cs, Tensor? sink, Tensor ext_off, Tensor seq_off, Tensor past, Tensor qt_seq, Tensor qt_start, Tensor(a!) y, int H, int D, int R, int V, float scale) -> ()", &latent_prompt_tc);
   m.def("linear_bias_residual(Tensor x, Tensor w, Tensor? bias, Tensor residual) -> Tensor", &linear_bias_residual);
   m.def("embedding_fwd(Tensor ids, Tensor table, int vocab_start) -> Tensor", &embedding_fwd);

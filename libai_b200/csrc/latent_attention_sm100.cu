@@ -12,7 +12,7 @@
 //                                TMEM, the output kept in TMEM and rescaled only when the running maximum grows by more than 2^8
 // Every wait on an mbarrier is bounded: when one runs out, the CTA stops issuing copies and products, runs its (finite) loops to
 // the end without waiting, lets the copies in flight land, frees its TMEM and reports through `err`.
-#include "common.cuh"
+#include "attention_tc.cuh"
 
 #include <type_traits>
 
@@ -40,23 +40,6 @@ struct LtcParams {
   float scale_log2;
   int* err;                  // mapped host word, set when a wait ran out
 };
-
-constexpr uint32_t LTC_WAIT_LIMIT = 1u << 22;
-LB_DEVICE bool ltc_wait(uint64_t* bar, uint32_t parity, volatile int* stop) {
-  if (*stop) return false;
-  for (uint32_t i = 0; i < LTC_WAIT_LIMIT; ++i) {
-    if (mbar_try_wait(bar, parity)) return true;
-    if ((i & 1023u) == 1023u && *stop) return false;
-  }
-  *stop = 1;
-  return false;
-}
-LB_DEVICE void ltc_pair_sync(int quad) {       // the two warps that own the same TMEM lane quadrant
-  if (quad == 0) asm volatile("bar.sync 1, 64;\n" ::: "memory");
-  else if (quad == 1) asm volatile("bar.sync 2, 64;\n" ::: "memory");
-  else if (quad == 2) asm volatile("bar.sync 3, 64;\n" ::: "memory");
-  else asm volatile("bar.sync 4, 64;\n" ::: "memory");
-}
 
 template <int DC, int V>
 __global__ void __launch_bounds__(LTC_THREADS, 1)
@@ -111,13 +94,13 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
       for (int j = 0; j < nkv; ++j) {
         const int s = j & 1, row = e0 + j * LTC_BN;
         const uint32_t par = ((j >> 1) & 1) ^ 1;
-        if (ltc_wait(&k_empty[s], par, stop)) {
+        if (tc_wait(&k_empty[s], par, stop)) {
           mbar_arrive_expect_tx(&k_full[s], Cfg::K_BYTES);
 #pragma unroll
           for (int c = 0; c < DC; ++c) tma_load_2d(sK + s * Cfg::K_BYTES + c * Cfg::CHUNK, &tmap_k, &k_full[s], head * (DC * 64) + c * 64, row);
           tma_load_2d(sK + s * Cfg::K_BYTES + DC * Cfg::CHUNK, &tmap_r, &k_full[s], 0, row);
         }
-        if (ltc_wait(&v_empty[s], par, stop)) {
+        if (tc_wait(&v_empty[s], par, stop)) {
           mbar_arrive_expect_tx(&v_full[s], Cfg::V_BYTES);
 #pragma unroll
           for (int c = 0; c < V / 64; ++c) tma_load_2d(sV + s * Cfg::V_BYTES + c * Cfg::CHUNK, &tmap_v, &v_full[s], head * V + c * 64, row);
@@ -130,12 +113,12 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
     constexpr uint32_t idesc_pv = make_idesc_bf16(LTC_BM, V, false, true);
     const uint32_t q_addr = smem_u32(sQ);
     const int rsteps = (p.R + 15) / 16;
-    bool ok = __all_sync(0xffffffffu, ltc_wait(q_ready, 0, stop));
+    bool ok = __all_sync(0xffffffffu, tc_wait(q_ready, 0, stop));
     // S(j + 1) is issued as soon as the softmax warps have read S(j) for the last time, ahead of P(j) V(j)
     auto issue_qk = [&](int j) {
       const int s = j & 1;
-      ok = __all_sync(0xffffffffu, ok && ltc_wait(&k_full[s], (j >> 1) & 1, stop));
-      if (j > 0) ok = __all_sync(0xffffffffu, ok && ltc_wait(s_free, (j - 1) & 1, stop));
+      ok = __all_sync(0xffffffffu, ok && tc_wait(&k_full[s], (j >> 1) & 1, stop));
+      if (j > 0) ok = __all_sync(0xffffffffu, ok && tc_wait(s_free, (j - 1) & 1, stop));
       tc_fence_after_sync();
       if (ok && elect_one()) {
         const uint32_t k_addr = smem_u32(sK + s * Cfg::K_BYTES);
@@ -156,8 +139,8 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
     for (int j = 0; j < nkv; ++j) {
       const int s = j & 1;
       if (j + 1 < nkv) issue_qk(j + 1);
-      ok = __all_sync(0xffffffffu, ok && ltc_wait(p_full, j & 1, stop));
-      ok = __all_sync(0xffffffffu, ok && ltc_wait(&v_full[s], (j >> 1) & 1, stop));
+      ok = __all_sync(0xffffffffu, ok && tc_wait(p_full, j & 1, stop));
+      ok = __all_sync(0xffffffffu, ok && tc_wait(&v_full[s], (j >> 1) & 1, stop));
       tc_fence_after_sync();
       if (ok && elect_one()) {
         const uint32_t v_addr = smem_u32(sV + s * Cfg::V_BYTES);
@@ -174,7 +157,7 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
     const int quad = warp_idx % 4, half = (warp_idx - 2) / 4;           // this warp's 64 of the 128 key columns
     const int r = quad * 32 + lane;                                     // query row of this thread (shared with the other half's thread)
     // ---- rotate the last query chunk in place: 16-byte unit u of row r sits at u ^ (r & 7)
-    ltc_wait(q_full, 0, stop);
+    tc_wait(q_full, 0, stop);
     if (r < nq) {
       uint8_t* row = sQ + DC * Cfg::CHUNK + r * 128;
       const float2* cs = p.cs + static_cast<long>(tok0 + r) * (p.R / 2);
@@ -201,7 +184,7 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
     float m_run = -INFINITY, l_run = 0.f;                               // log2 domain; l_run: the sum over this half's columns
     const int key_lim = pos0 + r + 1;                                   // keys [0, key_lim) are visible to this row
     for (int j = 0; j < nkv; ++j) {
-      ltc_wait(s_full, j & 1, stop);
+      tc_wait(s_full, j & 1, stop);
       __syncwarp();
       tc_fence_after_sync();
       const int k0 = j * LTC_BN + half * 64;
@@ -225,7 +208,7 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
       if (need_mask) pass1(std::true_type{}); else pass1(std::false_type{});
       float* xch = sXchg + (j & 1) * 256;
       xch[half * 128 + r] = mx;
-      ltc_pair_sync(quad);
+      tc_pair_sync(quad);
       mx = fmaxf(mx, xch[(half ^ 1) * 128 + r]);
       const float m_cand = fmaxf(m_run, mx * p.scale_log2);
       const bool bump = (m_cand - m_run > 8.0f) || (m_run == -INFINITY && m_cand != -INFINITY);
@@ -265,7 +248,7 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
         rowsum = rs0 + rs1;
       };
       // P(j) overwrites the columns that P(j - 1) V(j - 1) reads
-      if (j > 0) { ltc_wait(o_full, (j - 1) & 1, stop); __syncwarp(); tc_fence_after_sync(); }
+      if (j > 0) { tc_wait(o_full, (j - 1) & 1, stop); __syncwarp(); tc_fence_after_sync(); }
       if (need_mask) pass2(std::true_type{}); else pass2(std::false_type{});
       l_run = l_run * alpha + rowsum;
       if (bump_any) {                                                   // rare: P(j - 1) V(j - 1) has retired, rescale this half's columns
@@ -286,10 +269,10 @@ latent_prompt_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid
     }
     float* xch = sXchg + (nkv & 1) * 256;
     xch[half * 128 + r] = l_run;
-    ltc_pair_sync(quad);
+    tc_pair_sync(quad);
     l_run += xch[(half ^ 1) * 128 + r];
     if (p.sink) l_run += fast_exp2(p.sink[head] * 1.4426950408889634f - m_run);
-    ltc_wait(o_full, (nkv - 1) & 1, stop);
+    tc_wait(o_full, (nkv - 1) & 1, stop);
     __syncwarp();
     tc_fence_after_sync();
     const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;

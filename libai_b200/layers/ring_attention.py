@@ -140,6 +140,10 @@ class RingAttention(nn.Module):
         return y
 
     def forward(self, h, rb, bufs, shared=None):
-        parts = {name: KF.linear(h, w) for name, w in self.input_weights()}
+        proj = KF.linear(h, torch.cat([w for _, w in self.input_weights()], 0))         # keys and values: column slices of one matrix
+        parts, at = {}, 0
+        for name, w in self.input_weights():
+            parts[name] = proj[:, at:at + w.shape[0]]
+            at += w.shape[0]
         y = torch.empty(h.shape[0], self.mix_features, dtype=h.dtype, device=h.device)
         return KF.linear(self.mix(parts, rb, bufs, y, {} if shared is None else shared), self.o)

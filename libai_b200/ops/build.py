@@ -25,7 +25,7 @@ SO_PATH = os.path.join(ROOT, "_C.so")
 CUDA_HOME = os.environ.get("CUDA_HOME", "/usr/local/cuda")
 NVCC = os.path.join(CUDA_HOME, "bin", "nvcc")
 
-CU_SOURCES = ["gemm_sm100.cu", "norm.cu", "elementwise.cu", "attention_sm100.cu", "latent_attention_sm100.cu", "comm_kernels.cu"]
+CU_SOURCES = ["gemm_sm100.cu", "norm.cu", "elementwise.cu", "attention_sm100.cu", "latent_attention_sm100.cu", "masked_attention_sm100.cu", "comm_kernels.cu"]
 CPP_SOURCES = ["bindings.cpp", "symm_mem.cpp"]
 SEQ_SO_PATH = os.path.join(ROOT, "_C_seq.so")
 SEQ_CU_SOURCES = ["seq_mixers.cu"]

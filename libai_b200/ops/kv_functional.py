@@ -317,18 +317,30 @@ def _gated(o, gate_row, wide: bool, out_scale: float):
 
 def masked_attention(q, kmat, vmat, ext, gate, rb, y, H: int, G: int, D: int, V: int, window: int, chunk: int, keep: int,
                      scale: float, mma: bool = True, softcap: float = 0.0, sink: bool = False, gate_wide: bool = False,
-                     out_scale: float = 1.0, temp=None):
+                     out_scale: float = 1.0, temp=None, tc: Optional[bool] = None):
     """Grouped-query softmax attention of every packed query over the rows of the ext matrix (``kmat`` ``[rows, G·D]``,
     ``vmat`` ``[rows, G·V]``: column slices with one row stride) that its mask admits: position j ≤ i with
     ``j ≥ ⌊i/chunk⌋·chunk`` (``chunk > 0``) or ``j > i − window or j < keep`` (``window > 0``).  Head h of the result is
     multiplied by ``sigmoid(gate[t, h])`` when a gate is given (``gate_wide``: channel c of head h by
     ``sigmoid(gate[t, h·V + c])``) and by ``out_scale``.  ``softcap`` > 0: scaled scores pass through ``cap · tanh(s / cap)``;
     ``sink``: the softmax has one more entry of score 0 without a value; ``temp = (coef, every)``: the query at position p is
-    multiplied by ``1 + coef · ln(⌊(p + 1) / every⌋ + 1)``.  bf16 inputs with head sizes the tensor-core kernel is built for take it;
-    ``mma=False`` keeps them on the generic kernel (fp32 inputs always are)."""
+    multiplied by ``1 + coef · ln(⌊(p + 1) / every⌋ + 1)``.  bf16 inputs take the tcgen05 kernel where it is built for their sizes and
+    mask and the step is long enough (``tc`` decides otherwise), then the mma.sync kernel where that one is; ``mma=False`` keeps them on the
+    generic kernel (fp32 inputs always are)."""
     if _native(q):
         count_launch()
         coef, every = temp if temp else (0.0, 0.0)
+        if tc is None:
+            tc = mma and max(rb.lens) >= TC_MIN_TOKENS
+        if tc and tc_eligible(q, kmat, vmat, gate if gate_wide else None, y, D, V, keep, scale, softcap, sink, temp):
+            seq, start = rb.query_tiles(TC_QUERY_TILE, longest_first=True)
+            if seq.numel() <= 65535:
+                from . import load_ext
+
+                load_ext(required=True).masked_attention_tc(q, kmat, vmat, ext.ext_off, ext.nsink, ext.cstart, gate, bool(gate_wide), rb.seq_off, rb.past, seq,
+                                                            start, y, H, G, D, V, window, chunk, float(scale), float(out_scale), float(coef),
+                                                            float(every))
+                return y
         tiles = (None, None)
         if mma and q.dtype == torch.bfloat16 and mma_eligible(q, kmat, vmat, y, D, V) and (
                 gate is None or not gate_wide or (gate.data_ptr() % 4 == 0 and gate.stride(0) % 2 == 0 and V % 2 == 0)):
@@ -348,6 +360,18 @@ def masked_attention(q, kmat, vmat, ext, gate, rb, y, H: int, G: int, D: int, V:
 
 
 MMA_HEAD_SIZES = (32, 48, 64, 96, 128)       # head sizes (keys = values) the tensor-core prompt kernel is built for
+TC_QUERY_TILE = 128            # queries per block of the tcgen05 prompt kernel
+TC_MIN_TOKENS = 64             # a step whose longest sequence brings fewer tokens would leave most of its tile empty
+
+
+def tc_eligible(q, kmat, vmat, gate, y, D: int, V: int, keep: int, scale: float, softcap: float, sink: bool, temp) -> bool:
+    """bf16 prompt steps whose sizes and mask the tcgen05 prompt kernel is built for (no kept-first tokens, score cap or sink; ``gate``: a
+    gate per channel)."""
+    return (q.dtype == torch.bfloat16 and D % 16 == 0 and V % 16 == 0 and 16 <= D <= 128 and 16 <= V <= 128 and keep == 0 and scale > 0
+            and not softcap and not sink and (temp is None or temp[0] >= 0)
+            and all(t is None or (t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0) for t in (q, kmat, vmat, gate, y)))
+
+
 GROUPED_DECODE = True                      # single-token steps: the grouped split kernel where its sizes allow
 PAGE_DECODE_BLOCKS = 592                   # blocks a single-token step over pages is cut into (four per SM)
 

@@ -239,3 +239,10 @@ def random_weights(cfg, seed=0):
             t = t * 1.2 / math.sqrt(shape[-1])
         W[name] = t.to(torch.bfloat16).to(F64)
     return W
+
+
+def greedy(cfg, W, prompt, n):
+    toks = list(prompt)
+    for _ in range(n):
+        toks.append(int(forward(toks, W, cfg)[-1].argmax()))
+    return toks[len(prompt):]
