@@ -3,8 +3,9 @@ attention with chunk / kept-first window masks and mixture-of-experts feed-forwa
 (active) feed-forward size, and of Salizen (hyper-connection streams, linear-attention recurrences, sink-softmax window
 attention) beside Nefelorn, and of Zubarax (post-norm blocks, paged attention with mixed heads beside an HGRN2 recurrence,
 input-weighted experts) beside Salizen, and of Voduzen (latent attention over the whole past, norms on the sublayers' outputs,
-experts that may pass a token on) beside Bumodra and Zubarax, random weights, one GPU.
-``bench.py --serving [--serving-model nefelorn|salizen|zubarax|voduzen]`` prints the result
+experts that may pass a token on) beside Bumodra and Zubarax, and of Fogezen (chunked attention beside a matrix memory, attention over
+the whole past, norms before and after every sublayer) beside Salizen and Llama, random weights, one GPU.
+``bench.py --serving [--serving-model nefelorn|salizen|zubarax|voduzen|fogezen]`` prints the result
 as one JSON line; ``--serving-kernels`` adds device times of the individual kernels of one block at the same sizes with their
 roofline fractions.
 
@@ -903,11 +904,204 @@ def kernel_table_voduzen(s, batch, prompt):
     return {"peaks": src, "hbm_bytes_per_s": hbm, "bf16_flops": flops, "rows": rows}
 
 
+# ======================================================================================================================
+# Fogezen beside Salizen (window attention beside a linear recurrence) and Llama
+# ======================================================================================================================
+def fogezen_config(s):
+    """The sizes of :data:`NEFELORN_SIZES`: blocks alternate between chunked attention beside a matrix memory (chunks as long as the
+    windows of the other models, a state of half-size keys like Salizen's recurrence) and attention over the whole past; dense
+    feed-forwards."""
+    D, H = s["dim"], s["heads"]
+    heads = {"heads": H, "kv_heads": s["kv_heads"], "dim": D, "vdim": D, "scale": D ** -0.5}
+    par = {"left": dict(heads, mask={"size": s["reach"]}, rot={"dims": D, "base": 20000.0}), "right": {"heads": H, "dim": D // 2, "vdim": D, "gate_cap": 15.0}}
+    att = dict(heads, q_temp={"coef": 0.1, "every": 512})
+    mlp = {"kind": "dense", "ff": s["ff"]}
+    layers = [{"type": "attention", "mixer": att, "mlp": mlp} if i % 2 else {"type": "parallel", "mixer": par, "mlp": mlp} for i in range(s["blocks"])]
+    return dict(vocab=s["vocab"], width=s["width"], norm={"eps": 1e-6}, embedding={"scale": s["width"] ** 0.5}, residual_mult=0.5, layers=layers)
+
+
+def salizen_dense_config(s, prompt):
+    """Salizen with every block a parallel one with a dense feed-forward, one stream; windows alternate between ``reach`` and the prompt."""
+    cfg = salizen_config(dict(s))
+    blocks = []
+    for i in range(s["blocks"]):
+        blk = json.loads(json.dumps(cfg["layers"][0]))
+        if i % 2:
+            blk["mixer"]["left"]["mask"]["size"] = prompt + 64
+        blocks.append(blk)
+    return dict(cfg, layers=blocks, streams=1)
+
+
+@torch.no_grad()
+def throughput_fogezen(s, batch, prompt, new_tokens, steps, warmup):
+    from libai_b200.config import DictConfig
+    from libai_b200.layers._param import param_defaults
+    from libai_b200.models import FogezenForCausalLM, SalizenForCausalLM
+
+    ids = torch.randint(1, s["vocab"], (batch, prompt), generator=torch.Generator().manual_seed(0))
+    out = {}
+    for name, cls, cfg in (("fogezen", FogezenForCausalLM, fogezen_config(s)), ("salizen", SalizenForCausalLM, salizen_dense_config(s, prompt))):
+        with param_defaults(dtype=torch.bfloat16, device="cuda", seed=1):
+            model = cls(DictConfig(cfg)).eval().cuda()
+        _stateful_throughput(model, name, ids, batch, new_tokens, steps, warmup, out)
+        del model
+        torch.cuda.empty_cache()
+    llama = build_nefelorn_and_llama(s)[1]
+    dev_ids = ids.cuda()
+    out["llama_prefill_ms"] = _time(lambda: llama(dev_ids), warmup, steps)
+    a, d = llama.model.layers[0].self_attn.local_heads, llama.model.layers[0].self_attn.head_size
+    one = dev_ids[:, :1].contiguous()
+    llama.set_cache([(torch.randn(batch, a, prompt, d, device="cuda").to(torch.bfloat16),
+                      torch.randn(batch, a, prompt, d, device="cuda").to(torch.bfloat16)) for _ in range(s["blocks"])])
+    out["llama_decode_ms"] = _time(lambda: llama(one, use_cache=True), warmup, new_tokens)
+    llama.set_cache(None)
+    out["llama_prefill_tokens_per_s"] = batch * prompt / out["llama_prefill_ms"] * 1e3
+    out["llama_decode_tokens_per_s"] = batch / out["llama_decode_ms"] * 1e3
+    out["params_llama"] = sum(p.numel() for p in llama.parameters())
+    return out
+
+
+@torch.no_grad()
+def kernel_table_fogezen(s, batch, prompt):
+    """Device time of every kernel of a Fogezen block at these sizes (prefill rows = batch·prompt; decode rows = batch) beside the like
+    kernel of Salizen, Nefelorn or Llama, with the bytes / FLOPs the operation needs and the fraction of the measured roofline."""
+    from libai_b200.inference.ragged import RaggedBatch
+    from libai_b200.inference.state_cache import SequenceStateCache
+    from libai_b200.layers import DynamicTanh
+    from libai_b200.layers._param import param_defaults
+    from libai_b200.ops import functional as OF
+    from libai_b200.ops import kv_functional as KF
+    from libai_b200.ops import lin_functional as LF
+    from libai_b200.ops import paged_functional as PF
+
+    hbm, flops, src = _peaks()
+    dev, bf = "cuda", torch.bfloat16
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    n, H, G, D, reach, ff = s["width"], s["heads"], s["kv_heads"], s["dim"], s["reach"], s["ff"]
+    Dm, C = D // 2, G * 2 * D
+    rows = []
+
+    def add(name, fn, bytes_=0.0, fl=0.0):
+        ms = _time(fn, flush=flush)
+        ideal = max(bytes_ / hbm, fl / flops) * 1e3
+        rows.append(dict(kernel=name, ms=round(ms, 4), ideal_ms=round(ideal, 5), roofline_fraction=round(ideal / ms, 4),
+                         bound="memory" if bytes_ / hbm >= fl / flops else "tensor"))
+
+    rnd = lambda *shape: torch.randn(*shape, device=dev).to(bf)
+    with param_defaults(dtype=bf, device=dev, seed=2):
+        na, nb = DynamicTanh(n), DynamicTanh(n)
+    cache = SequenceStateCache(dev, bf, max_slots=batch, page_size=64)
+    paged = cache.register("paged", channels=C, taps=1, conv_channels=0)
+    mem = cache.register("recurrent", heads=H, dim=Dm, vdim=D, taps=1, conv_channels=0, peaks=True)
+    slots = cache.allocate(batch)
+    cache.prepare(slots, [prompt + 1] * batch)
+    pages, state = cache.buffers(paged), cache.buffers(mem)
+    pages["pool"].copy_(rnd(*pages["pool"].shape))
+    freq, nofreq = KF.rotary_frequencies(D, 2e4)[0].to(dev), torch.zeros(0, device=dev)
+    half = KF.rotary_frequencies(D // 2, 1e6)[0].to(dev)
+    w, wd = torch.zeros(n, dtype=bf, device=dev), torch.ones(D, dtype=bf, device=dev)
+    wm, zb = torch.ones(H * D, dtype=bf, device=dev), torch.zeros(2 * H, device=dev)
+    temp = (0.1, 512.0)
+    for phase, lens, past in (("prefill", [prompt] * batch, [0] * batch), ("decode", [1] * batch, [prompt] * batch)):
+        rb = RaggedBatch(lens, slots, past, dev)
+        T = rb.tokens
+        x, y1, y2, h = torch.randn(T, n, device=dev), torch.randn(T, n, device=dev), torch.randn(T, n, device=dev), torch.empty(T, n, dtype=bf, device=dev)
+        add(f"{phase}: closing norm + scaled residual + opening norm", lambda: PF.sandwich_residual(x, 1e-6, y=y1, post=w, mult=0.5, nxt=w, h=h), T * n * 14)
+        add(f"{phase}: the same with two normed branches and the row that enters a pass",
+            lambda: PF.sandwich_residual(x, 1e-6, y=y1, post=w, mult=0.5, y2=y2, branch=(w, w), add=w, nxt=w, h=h), T * n * 18)
+        add(f"{phase}: Nefelorn closing norm + residual + opening norm (Dynamic Tanh)", lambda: KF.dyt_residual(x, y1, post=na.triple(), nxt=nb.triple(), h=h), T * n * 14)
+        qkv = rnd(T, H * D + C)
+        q, k, v = qkv[:, :H * D], qkv[:, H * D:H * D + G * D], qkv[:, H * D + G * D:]
+        ring, first = torch.zeros(batch, reach, C, dtype=bf, device=dev), torch.zeros(batch, 0, C, dtype=bf, device=dev)
+        long_ring = torch.randn(batch, prompt + 64, C, device=dev).to(bf)
+        kept = min(T, batch * reach)
+        add(f"{phase}: head norms + rotation of q, k + ring write", lambda: KF.heads_prepare(q, k, v, wd, wd, freq, 1e-6, rb, H, G, D, D, ring=ring),
+            T * (H * D + G * D) * 4 + kept * C * 2 + T * G * D * 2)
+        add(f"{phase}: page write of k, v", lambda: KF.heads_prepare(q, k, v, None, None, nofreq, 1e-6, rb, H, G, D, D, pool=pages["pool"], table=pages["table"]), T * C * 4)
+
+        def salizen_prepare():
+            KF.qk_prepare(q, k, None, None, half, 1.0, rb, H, G, D, 1e-6, False, False)
+            KF.kv_write(ring, first, k, v, rb)
+
+        add(f"{phase}: Salizen rotation of q, k + ring write (two kernels, no norms)", salizen_prepare, T * (H * D + G * D) * 4 + kept * C * 4)
+        gate, yb = rnd(T, H * D), torch.empty(T, H * D, dtype=bf, device=dev)
+        io = T * H * D * 4 + T * C * 2
+        if phase == "prefill":
+            full = prompt * (prompt + 1) // 2 * batch
+            inside = sum(p % reach + 1 for p in range(prompt)) * batch
+            window = sum(min(p + 1, reach) for p in range(prompt)) * batch
+            ext = rb.kv_ext([(0, 0, 0)])
+            for name, kw in (("tcgen05", dict(tc=True)), ("mma.m16n8k16, for other head sizes", dict(tc=False))):
+                add(f"prefill: attention over the whole past, query temperature ({name})",
+                    lambda: KF.masked_attention(q, k, v, ext, None, rb, yb, H, G, D, D, 0, 0, 0, D ** -0.5, temp=temp, **kw), io, full * H * D * 4.0)
+            qkv4 = rnd(batch, prompt, H, 3 * D)
+            add("prefill: Llama causal flash attention, same query heads (tcgen05)", lambda: OF.attention_qkvpacked(qkv4, causal=True, scale=D ** -0.5),
+                qkv4.numel() * 2 + T * H * D * 2, full * H * D * 4.0)
+            cext, wext = rb.kv_ext([(0, reach, 0)]), rb.kv_ext([(reach, 0, 0)])
+            for name, kw in (("tcgen05", dict(tc=True)), ("mma.m16n8k16, for other head sizes", dict(tc=False))):
+                add(f"prefill: chunked attention with channel gate ({name})",
+                    lambda: KF.masked_attention(q, k, v, cext, gate, rb, yb, H, G, D, D, 0, reach, 0, D ** -0.5, gate_wide=True, **kw), io + T * H * D * 2,
+                    inside * H * D * 4.0)
+            add("prefill: Salizen window attention with cap, sink, channel gate (mma.m16n8k16)",
+                lambda: KF.masked_attention(q, k, v, wext, gate, rb, yb, H, G, D, D, reach, 0, 0, D ** -0.5, gate_wide=True, softcap=30.0, sink=True),
+                io + T * H * D * 2, window * H * D * 4.0)
+        else:
+            add("decode: attention over the pages, query temperature (keys in parts + merge)",
+                lambda: KF.page_attention(q, pages["pool"], pages["table"], None, rb, yb, H, G, D, D, D ** -0.5, temp=temp), batch * (prompt + 1) * C * 2)
+            add("decode: Salizen grouped ring attention with cap and sink, window = prompt",
+                lambda: KF.ring_attention(q, long_ring, first, None, rb, yb, H, G, D, D, prompt + 64, 0, 0, D ** -0.5, softcap=30.0, sink=True),
+                batch * (prompt + 1) * C * 2)
+            last = RaggedBatch([1] * batch, slots, [prompt - 1] * batch, dev)         # the last position of a chunk: a whole chunk is visible
+            add("decode: chunked attention with channel gate over the ring",
+                lambda: KF.ring_attention(q, ring, first, gate, last, yb, H, G, D, D, 0, reach, 0, D ** -0.5, gate_wide=True), batch * reach * C * 2)
+            add("decode: Salizen window attention over its ring (cap, sink, channel gate)",
+                lambda: KF.ring_attention(q, ring, first, gate, last, yb, H, G, D, D, reach, 0, 0, D ** -0.5, gate_wide=True, softcap=30.0, sink=True),
+                batch * reach * C * 2)
+        qm, km, vm, z = rnd(T, H * Dm), rnd(T, H * Dm), rnd(T, H * D), torch.randn(T, 2 * H, device=dev)
+        hb, wz = rnd(T, n), rnd(2 * H, n)
+        zc, zcb, S2 = torch.randn(T, H * Dm, device=dev), torch.randn(H * Dm, device=dev) + 2.0, torch.zeros(batch, H, Dm, D, device=dev)
+        st = batch * H * Dm * D * 4 * (2 if phase == "decode" else 1)
+        add(f"{phase}: gate logits of the memory (fp32 product)", lambda: KF.router_logits(hb, wz), T * n * 2)
+        if phase == "prefill":
+            add(f"prefill: matrix memory (gates, then the recurrence; state {Dm} x {D})",
+                lambda: LF.memory_scan(qm, km, vm, z, zb, H, 15.0, Dm ** -0.5, state, rb), T * H * (Dm * 4 + D * 6 + 8) + st)
+            o = torch.randn(T, H * D, device=dev)
+            add("prefill: RMS norm per head, weight, sigmoid gate", lambda: LF.gated_norm(o, gate, wm, 1e-6, LF.GATE_SIGMOID, yb, H, D, per_head=True), T * H * D * 8)
+            add("prefill: Salizen gated RMS norm per head", lambda: LF.gated_norm(o, gate, wd, 1e-6, LF.GATE_SILU, yb, H, D, per_head=True), T * H * D * 8)
+            add(f"prefill: Salizen decay scan, decay logits per key channel (state {Dm} x {D})",
+                lambda: LF.decay_scan(qm, km, vm, S2, rb, z=zc, zb=zcb, tau=8.0, q_scale=Dm ** -0.5), T * H * (Dm * 8 + D * 6) + st)
+            gu, a = rnd(T, 2 * ff), torch.empty(T, ff, dtype=bf, device=dev)
+            add("prefill: gated tanh-GELU of the feed-forward (Salizen's kernel)", lambda: KF.act_rows(gu, a, KF.ACTS["gelu_tanh"], gated=True), T * ff * 6)
+        else:
+            add("decode: matrix memory, one kernel (gates, state, read-out, norm, gate)",
+                lambda: LF.memory_step(qm, km, vm, z, zb, H, 15.0, Dm ** -0.5, state, rb, wm, gate, 1e-6, yb), T * H * (Dm * 4 + D * 6) + st)
+
+            def salizen_step():
+                LF.gated_norm(LF.decay_scan(qm, km, vm, S2, rb, z=zc, zb=zcb, tau=8.0, q_scale=Dm ** -0.5), gate, wd, 1e-6, LF.GATE_SILU, yb, H, D, per_head=True)
+
+            add("decode: Salizen decay scan + gated norm (two kernels)", salizen_step, T * H * (Dm * 8 + D * 6) + st)
+    return {"peaks": src, "hbm_bytes_per_s": hbm, "bf16_flops": flops, "rows": rows}
+
+
 def main(args):
     assert torch.cuda.is_available(), "the serving bench needs a GPU"
     from libai_b200 import ops
 
     ops.reset_launch_count()
+    if getattr(args, "serving_model", "bumodra") == "fogezen":
+        result = {"metric": "prefill / decode tokens per second, Fogezen beside Salizen (parallel blocks, dense feed-forward, one stream, the same reaches) and Llama at equal width, depth, heads and feed-forward size",
+                  "dtype": "bf16", "data": "synthetic tokens, random-init weights", "n_gpus": 1, "sizes": {}}
+        for name in (args.serving_sizes.split(",") if args.serving_sizes else list(NEFELORN_SIZES)):
+            s = NEFELORN_SIZES[name]
+            r = throughput_fogezen(s, args.serving_batch, args.serving_prompt, new_tokens=max(args.steps, 8),
+                                   steps=max(args.steps // 2, 3), warmup=max(args.warmup, 3))
+            if args.serving_kernels:
+                r["kernels"] = kernel_table_fogezen(s, args.serving_batch, args.serving_prompt)
+            result["sizes"][name] = {"config": dict(s), "batch": args.serving_batch, "prompt": args.serving_prompt, **r}
+            torch.cuda.empty_cache()
+        result["gpu_launches"] = ops.launch_count()
+        print(json.dumps(result))
+        return
     if getattr(args, "serving_model", "bumodra") == "voduzen":
         result = {"metric": "prefill / decode tokens per second, Voduzen beside Bumodra (latent attention, window = prompt, dense feed-forward of the active size) and Zubarax (paged attention, experts) at equal width, depth and heads",
                   "dtype": "bf16", "data": "synthetic tokens, random-init weights", "n_gpus": 1, "sizes": {}}
