@@ -18,7 +18,11 @@ int lbl_decay_scan(const void* q, long ldq, const void* k, long ldk, const void*
                    const int* seq_off, const int* slots, const int* past, float* out, int B, int H, int D, int V, int dtype,
                    cudaStream_t s);
 int lbl_memory_gates(const float* z, long ldz, int foff, const float* zb, float cap, float* mx, const int* seq_off, const int* slots,
-                     const int* past, float* gates, long tokens, int B, int H, cudaStream_t s);
+                     const int* past, float* gates, long tokens, int B, int H, int chunk, cudaStream_t s);
+int lbm_memory_chunk_blocks(const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, int B, int H, int D, int V);
+int lbm_memory_chunk(const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, const float* gates, float q_scale, float* S,
+                     float* Z, float* ztmp, const int* seq_off, const int* slots, const int* past, float* out, const void* w, const void* gate,
+                     long ldg, float eps, float out_scale, void* y, long ldy, long tokens, int B, int H, int D, int V, int blocks, cudaStream_t s);
 int lbl_memory_scan(const void* q, long ldq, const void* k, long ldk, const void* v, long ldv, const float* gates, float q_scale, float* S,
                     float* Z, float* ztmp, const int* seq_off, const int* slots, const int* past, float* out, long tokens, int B, int H, int D, int V,
                     int dtype, cudaStream_t s);
@@ -174,10 +178,47 @@ void memory_scan(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor
   const int B = (int)slots.numel();
   Tensor gates = at::empty({m.H, 3, tokens}, z.options()), ztmp = at::empty({B, m.H, m.D}, z.options());
   check(lbl_memory_gates(z.data_ptr<float>(), z.stride(0), (int)foff, zb.data_ptr<float>(), (float)cap, mx.data_ptr<float>(), meta(seq_off), meta(slots),
-                         meta(past), gates.data_ptr<float>(), tokens, B, m.H, cur_stream()), "memory_gates");
+                         meta(past), gates.data_ptr<float>(), tokens, B, m.H, 0, cur_stream()), "memory_gates");
   check(lbl_memory_scan(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), gates.data_ptr<float>(), (float)q_scale,
                         S.data_ptr<float>(), Z.data_ptr<float>(), ztmp.data_ptr<float>(), meta(seq_off), meta(slots), meta(past), out.data_ptr<float>(), tokens, B, m.H, m.D,
                         m.V, code(q), cur_stream()), "memory_scan");
+}
+
+// into how many blocks of value columns per head the chunked form would cut these operands (0: it does not take them)
+int64_t memory_chunk_blocks(const Tensor& q, const Tensor& k, const Tensor& v, int64_t B, int64_t H, int64_t D, int64_t V) {
+  if (q.scalar_type() != at::kBFloat16 || k.scalar_type() != at::kBFloat16 || v.scalar_type() != at::kBFloat16) return 0;
+  return lbm_memory_chunk_blocks(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), (int)B, (int)H, (int)D, (int)V);
+}
+
+// the chunked form (bf16): out fp32 [tokens, H*V], or — one block of columns only — y bf16 [tokens, H*V], the normed, weighted, gated read-out
+void memory_chunks(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& z, const Tensor& zb, int64_t foff, double cap, double q_scale,
+                   Tensor S, Tensor Z, Tensor mx, const Tensor& seq_off, const Tensor& slots, const Tensor& past, const OptT& out, const OptT& w,
+                   const OptT& gate, double eps, double out_scale, const OptT& y) {
+  const MemoryShape m = memory_state(S, Z, mx);
+  memory_operands(q, k, v, z, zb, foff, m);
+  const int64_t tokens = q.size(0);
+  const int B = (int)slots.numel();
+  const int blocks = (int)memory_chunk_blocks(q, k, v, B, m.H, m.D, m.V);
+  TORCH_CHECK(blocks > 0, "memory_chunks: bf16 operands of sizes and alignments the kernel is built for");
+  TORCH_CHECK(has(out) != has(y) && (!has(y) || blocks == 1), "memory_chunks: one of out and y (y with one block of columns)");
+  if (has(out)) TORCH_CHECK(out->is_cuda() && out->scalar_type() == at::kFloat && out->is_contiguous() && out->dim() == 2 && out->size(0) == tokens && out->size(1) == (long)m.H * m.V, "memory_chunks: out fp32 [tokens, H*V]");
+  long ldg = 0, ldy = 0;
+  if (has(y)) {
+    rows2d(*y, "memory_chunks y");
+    TORCH_CHECK(y->scalar_type() == at::kBFloat16 && y->size(0) == tokens && y->size(1) == (long)m.H * m.V, "memory_chunks: y bf16 [tokens, H*V]");
+    ldy = y->stride(0);
+    if (has(gate)) { rows2d(*gate, "memory_chunks gate"); TORCH_CHECK(gate->scalar_type() == at::kBFloat16 && gate->size(0) == tokens && gate->size(1) == y->size(1), "memory_chunks: gate [tokens, H*V]"); ldg = gate->stride(0); }
+    if (has(w)) TORCH_CHECK(w->is_cuda() && w->is_contiguous() && w->numel() == y->size(1) && w->scalar_type() == at::kBFloat16, "memory_chunks: weight [H*V]");
+  }
+  c10::cuda::CUDAGuard guard(q.device());
+  Tensor gates = at::empty({m.H, 6, tokens}, z.options()), ztmp = at::empty({blocks > 1 ? B : 0, m.H, m.D}, z.options());
+  check(lbl_memory_gates(z.data_ptr<float>(), z.stride(0), (int)foff, zb.data_ptr<float>(), (float)cap, mx.data_ptr<float>(), meta(seq_off), meta(slots),
+                         meta(past), gates.data_ptr<float>(), tokens, B, m.H, 64, cur_stream()), "memory_gates");
+  check(lbm_memory_chunk(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), gates.data_ptr<float>(), (float)q_scale,
+                         S.data_ptr<float>(), Z.data_ptr<float>(), ztmp.data_ptr<float>(), meta(seq_off), meta(slots), meta(past),
+                         has(out) ? out->data_ptr<float>() : nullptr, has(w) && has(y) ? w->data_ptr() : nullptr, has(gate) && has(y) ? gate->data_ptr() : nullptr,
+                         ldg, (float)eps, (float)out_scale, has(y) ? y->data_ptr() : nullptr, ldy, tokens, B, m.H, m.D, m.V, blocks, cur_stream()),
+        "memory_chunks");
 }
 
 // one token per sequence, through to the gated, normed read-out y [tokens, H*V]
@@ -205,5 +246,7 @@ TORCH_LIBRARY(libai_b200_lin, m) {
   m.def("decay_scan(Tensor q, Tensor k, Tensor v, Tensor? decay, Tensor? z, Tensor? zb, float inv_tau, float q_scale, float k_scale, int act, Tensor(a!) S, Tensor seq_off, Tensor slots, Tensor past, Tensor(b!) out, Tensor? lower=None) -> ()", &decay_scan);
   m.def("gated_norm(Tensor o, Tensor? gate, Tensor? w, float eps, int act, float out_scale, Tensor(a!) y, int H, int V, bool per_head, bool wide=False) -> ()", &gated_norm);
   m.def("memory_scan(Tensor q, Tensor k, Tensor v, Tensor z, Tensor zb, int foff, float cap, float q_scale, Tensor(a!) S, Tensor(b!) Z, Tensor(c!) mx, Tensor seq_off, Tensor slots, Tensor past, Tensor(d!) out) -> ()", &memory_scan);
+  m.def("memory_chunk_blocks(Tensor q, Tensor k, Tensor v, int B, int H, int D, int V) -> int", &memory_chunk_blocks);
+  m.def("memory_chunks(Tensor q, Tensor k, Tensor v, Tensor z, Tensor zb, int foff, float cap, float q_scale, Tensor(a!) S, Tensor(b!) Z, Tensor(c!) mx, Tensor seq_off, Tensor slots, Tensor past, Tensor(d!)? out, Tensor? w, Tensor? gate, float eps, float out_scale, Tensor(e!)? y) -> ()", &memory_chunks);
   m.def("memory_step(Tensor q, Tensor k, Tensor v, Tensor z, Tensor zb, int foff, float cap, float q_scale, Tensor(a!) S, Tensor(b!) Z, Tensor(c!) mx, Tensor slots, Tensor past, Tensor? w, Tensor? gate, float eps, float out_scale, Tensor(d!) y) -> ()", &memory_step);
 }

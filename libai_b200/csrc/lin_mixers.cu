@@ -505,7 +505,9 @@ decay_scan_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, lo
 //   S <- decay S + write k v^T,   z <- decay z + write k,   o = S^T q / (max(|z q|, floor) + 1e-6).
 // memory_gates_kernel: one warp per (sequence, head) turns the logits of the step into gates [H][3][tokens] = decay, write, floor, 32 tokens
 // at a time: with F_t = sum of f over the group, m_t = max(F_t + m_in, max_s (i_s + F_t - F_s)) is a scan of (f, i) pairs under
-// (F1 + F2, max(M1 + F2, M2)).  mx [slots, H] holds the running maximum between steps.
+// (F1 + F2, max(M1 + F2, M2)).  mx [slots, H] holds the running maximum between steps.  `chunk` > 0 (a multiple of 32): gates
+// [H][6][tokens] instead, for the chunked form (memory_mixers.cu): F from the chunk's start in two numbers (upper part and rest, so that
+// differences keep their digits), i, m, exp(F + m before the chunk - m), exp(-m).
 // ------------------------------------------------------------------------------------------------------------------
 __device__ __forceinline__ void memory_log_gates(float zi, float zf, float cap, float& li, float& lf) {
   li = cap * tanhf(zi / cap);
@@ -517,9 +519,16 @@ __global__ void memory_keysum_kernel(const float* __restrict__ ztmp, float* __re
   for (int i = threadIdx.x; i < D; i += blockDim.x) Z[((long)slots[b] * H + h) * D + i] = ztmp[(long)blockIdx.x * D + i];
 }
 
+// (h, l) += (ph, pl), the rounding error of the upper parts' sum kept in l
+__device__ __forceinline__ void add_exact(float& h, float& l, float ph, float pl) {
+  const float s = h + ph, t = s - h;
+  l = l + pl + ((h - (s - t)) + (ph - t));
+  h = s;
+}
+
 __global__ void memory_gates_kernel(const float* __restrict__ z, long ldz, int foff, const float* __restrict__ zb, float cap,
                                     float* __restrict__ mx, const int* __restrict__ seq_off, const int* __restrict__ slots,
-                                    const int* __restrict__ past, float* __restrict__ gates, long tokens, int B, int H) {
+                                    const int* __restrict__ past, float* __restrict__ gates, long tokens, int B, int H, int chunk) {
   const int wid = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (wid >= B * H) return;
   const int b = wid / H, h = wid - b * H;
@@ -528,21 +537,34 @@ __global__ void memory_gates_kernel(const float* __restrict__ z, long ldz, int f
   float* mslot = mx + (long)slots[b] * H + h;
   float m = past[b] > 0 ? *mslot : 0.f;
   const float bi = zb[h], bf = zb[foff + h];
-  float* g0 = gates + (long)h * 3 * tokens + tok0;
+  float* g0 = gates + (long)h * (chunk ? 6 : 3) * tokens + tok0;
+  float Ch = 0.f, Cl = 0.f, m0 = m;               // F of the chunk so far, m before the chunk
   for (int t0 = 0; t0 < n; t0 += 32) {
     const int t = t0 + lane;
     float li = -INFINITY, lf = 0.f;               // beyond the end: the maximum stays
     if (t < n) memory_log_gates(z[(tok0 + t) * ldz + h] + bi, z[(tok0 + t) * ldz + foff + h] + bf, cap, li, lf);
-    float F = lf, M = li;
+    float F = lf, Fl = 0.f, M = li;
 #pragma unroll
     for (int d = 1; d < 32; d <<= 1) {
-      const float Fp = __shfl_up_sync(0xffffffffu, F, d), Mp = __shfl_up_sync(0xffffffffu, M, d);
-      if (lane >= d) { M = fmaxf(Mp + F, M); F += Fp; }
+      const float Fp = __shfl_up_sync(0xffffffffu, F, d), Flp = __shfl_up_sync(0xffffffffu, Fl, d), Mp = __shfl_up_sync(0xffffffffu, M, d);
+      if (lane >= d) { M = fmaxf(Mp + F, M); add_exact(F, Fl, Fp, Flp); }
     }
     const float mt = fmaxf(F + m, M);
     float mp = __shfl_up_sync(0xffffffffu, mt, 1);
     if (lane == 0) mp = m;
-    if (t < n) {
+    if (chunk) {
+      if (t0 % chunk == 0) { Ch = Cl = 0.f; m0 = m; }
+      add_exact(F, Fl, Ch, Cl);
+      Ch = __shfl_sync(0xffffffffu, F, 31); Cl = __shfl_sync(0xffffffffu, Fl, 31);
+      if (t < n) {
+        g0[t] = F;
+        g0[tokens + t] = Fl;
+        g0[2 * tokens + t] = li;
+        g0[3 * tokens + t] = mt;
+        g0[4 * tokens + t] = expf((F + (m0 - mt)) + Fl);
+        g0[5 * tokens + t] = expf(-mt);
+      }
+    } else if (t < n) {
       g0[t] = expf(lf + mp - mt);
       g0[tokens + t] = expf(li - mt);
       g0[2 * tokens + t] = expf(-mt);
@@ -808,10 +830,10 @@ int lbl_decay_scan(const void* q, long ldq, const void* k, long ldk, const void*
 }
 
 int lbl_memory_gates(const float* z, long ldz, int foff, const float* zb, float cap, float* mx, const int* seq_off, const int* slots,
-                     const int* past, float* gates, long tokens, int B, int H, cudaStream_t s) {
+                     const int* past, float* gates, long tokens, int B, int H, int chunk, cudaStream_t s) {
   if (B == 0 || tokens == 0) return 0;
-  if (!(cap > 0.f)) return -1;
-  memory_gates_kernel<<<(unsigned)((B * H + 3) / 4), 128, 0, s>>>(z, ldz, foff, zb, cap, mx, seq_off, slots, past, gates, tokens, B, H);
+  if (!(cap > 0.f) || chunk % 32) return -1;
+  memory_gates_kernel<<<(unsigned)(B * H), 32, 0, s>>>(z, ldz, foff, zb, cap, mx, seq_off, slots, past, gates, tokens, B, H, chunk);
   LAUNCH_END();
 }
 

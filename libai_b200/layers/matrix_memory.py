@@ -13,8 +13,9 @@ Every head's ``o`` is divided by its root mean square, the heads are concatenate
 
 The gates (their logits leave the product in fp32), the recurrence, the norm and the output gate's activation are fp32 in every compute
 dtype.  State per sequence (:class:`libai_b200.inference.state_cache.SequenceStateCache`, kind ``recurrent`` with ``peaks``): ``S``, the sums
-``z`` and ``m``.  Prompt steps turn the logits into decay, write weight and floor of every token (a scan of pairs), then run the
-recurrence; single-token steps are one kernel from the projections to the input of ``W_o``.
+``z`` and ``m``.  Prompt steps turn the logits into what the recurrence needs per token (a scan of pairs), then run it: chunk by
+chunk on the tensor cores in bf16, through the norm and the gate, or token by token; single-token steps are one kernel from the
+projections to the input of ``W_o``.
 """
 from __future__ import annotations
 
@@ -74,8 +75,7 @@ class MatrixMemory(nn.Module):
         q, k, v, g = parts["q"], parts["k"], parts["v"], parts["g"]
         if rb.single:
             return LF.memory_step(q, k, v, z, b, foff, self.gate_cap, self.q_scale, bufs, rb, self.norm, g, self.eps, y, out_scale)
-        o = LF.memory_scan(q, k, v, z, b, foff, self.gate_cap, self.q_scale, bufs, rb)
-        return LF.gated_norm(o, g, self.norm, self.eps, LF.GATE_SIGMOID, y, self.heads, self.vdim, per_head=True, out_scale=out_scale)
+        return LF.memory_prompt(q, k, v, z, b, foff, self.gate_cap, self.q_scale, bufs, rb, self.norm, g, self.eps, y, out_scale)
 
     def forward(self, h, rb, bufs):
         """Unfused form: ``h`` ``[tokens, width]`` packed rows → ``[tokens, width]``."""

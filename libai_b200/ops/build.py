@@ -1,7 +1,7 @@
 """In-tree build of the native extensions: ``libai_b200/_C.so`` (GEMM, attention, norms, optimizer, collectives) and
 ``libai_b200/_C_seq.so`` (ragged-batch sequence mixers with per-sequence state), ``libai_b200/_C_kv.so`` (ring and paged key/value
 caches, masked grouped-query attention, attention with mixed heads, attention on paged latents, Dynamic-Tanh and post-norm residuals, mixture of experts) and ``libai_b200/_C_lin.so`` (bigram embedding,
-hyper-connection streams, decayed linear-attention recurrences).
+hyper-connection streams, decayed linear-attention recurrences, matrix memory with exponential gates).
 
     python -m libai_b200.ops.build [--force] [--verbose] [--only _C|_C_seq|_C_kv|_C_lin]
 
@@ -34,7 +34,7 @@ KV_SO_PATH = os.path.join(ROOT, "_C_kv.so")
 KV_CU_SOURCES = ["kv_mixers.cu", "paged_mixers.cu", "latent_mixers.cu"]
 KV_CPP_SOURCES = ["kv_bindings.cpp", "latent_bindings.cpp"]
 LIN_SO_PATH = os.path.join(ROOT, "_C_lin.so")
-LIN_CU_SOURCES = ["lin_mixers.cu"]
+LIN_CU_SOURCES = ["lin_mixers.cu", "memory_mixers.cu"]
 LIN_CPP_SOURCES = ["lin_bindings.cpp"]
 
 NVCC_FLAGS = [

@@ -124,17 +124,22 @@ def memory_gates(z, zb, foff: int, cap: float, H: int):
     return u[:, :H], F.logsigmoid(u[:, foff:foff + H])
 
 
-def memory_scan(q, k, v, z, zb, foff: int, cap: float, q_scale: float, bufs, rb):
+def memory_scan(q, k, v, z, zb, foff: int, cap: float, q_scale: float, bufs, rb, chunks: bool = True):
     """The matrix memory with exponential gates over the packed rows (``q``, ``k`` ``[tokens, H·D]``, ``v`` ``[tokens, H·V]``): with the
     log gates ``i``, ``f`` of :func:`memory_gates` and a running maximum ``m`` (0 at the start of a sequence),
     ``m' = max(f + m, i)``, ``S ← e^(f+m−m') S + e^(i−m') k vᵀ``, ``z ← …`` likewise with ``k`` alone, and the read-out is
     ``Sᵀq / (max(|z·q|, e^(−m')) + 1e-6)``.  ``bufs``: ``S`` ``[slots, H, D, V]``, ``keys`` (the sums ``z``) ``[slots, H, D]`` and ``peak`` (``m``)
-    ``[slots, H]``, all fp32; they are read unless ``past == 0`` and left at the state after the last row.  Returns fp32 ``[tokens, H·V]``."""
+    ``[slots, H]``, all fp32; they are read unless ``past == 0`` and left at the state after the last row.  Returns fp32 ``[tokens, H·V]``.  bf16 operands
+    of suitable sizes run chunk by chunk on the tensor cores; ``chunks=False`` keeps them on the token-by-token kernel (fp32 always is)."""
     S, Z, mx = bufs["S"], bufs["keys"], bufs["peak"]
     H, D, V = S.shape[1:]
     out = torch.empty(q.shape[0], H * V, dtype=torch.float32, device=q.device)
     if _native(q):
         count_launch(2)
+        if chunks and load_lin_ext().memory_chunk_blocks(q, k, v, rb.B, H, D, V):
+            load_lin_ext().memory_chunks(q, k, v, z, zb, int(foff), float(cap), float(q_scale), S, Z, mx, rb.seq_off, rb.slots, rb.past, out, None,
+                                         None, 0.0, 1.0, None)
+            return out
         load_lin_ext().memory_scan(q, k, v, z, zb, int(foff), float(cap), float(q_scale), S, Z, mx, rb.seq_off, rb.slots, rb.past, out)
         return out
     li, lf = memory_gates(z, zb, foff, cap, H)
@@ -157,6 +162,21 @@ def memory_scan(q, k, v, z, zb, foff: int, cap: float, q_scale: float, bufs, rb)
     return out
 
 
+def memory_prompt(q, k, v, z, zb, foff: int, cap: float, q_scale: float, bufs, rb, w, gate, eps: float, y, out_scale: float = 1.0):
+    """Prompt steps: :func:`memory_scan`, then every head divided by its root mean square, times ``w`` ``[H·V]``, ``sigmoid(gate)`` and
+    ``out_scale``, into ``y`` ``[tokens, H·V]``.  The chunked form does it all in one kernel where one block holds a head's values."""
+    S = bufs["S"]
+    H, D, V = S.shape[1:]
+    if (_native(q) and y.dtype == torch.bfloat16 and load_lin_ext().memory_chunk_blocks(q, k, v, rb.B, H, D, V) == 1
+            and all(t is None or (t.data_ptr() % 4 == 0 and (t.dim() == 1 or t.stride(0) % 2 == 0)) for t in (y, gate, w))):
+        count_launch(2)
+        load_lin_ext().memory_chunks(q, k, v, z, zb, int(foff), float(cap), float(q_scale), S, bufs["keys"], bufs["peak"], rb.seq_off, rb.slots,
+                                     rb.past, None, w, gate, float(eps), float(out_scale), y)
+        return y
+    o = memory_scan(q, k, v, z, zb, foff, cap, q_scale, bufs, rb)
+    return gated_norm(o, gate, w, eps, GATE_NONE if gate is None else GATE_SIGMOID, y, H, V, per_head=True, out_scale=out_scale)
+
+
 def memory_step(q, k, v, z, zb, foff: int, cap: float, q_scale: float, bufs, rb, w, gate, eps: float, y, out_scale: float = 1.0):
     """Single-token steps in one kernel: :func:`memory_scan`, then every head divided by its root mean square, times ``w`` ``[H·V]``,
     ``sigmoid(gate)`` and ``out_scale``, into ``y`` ``[tokens, H·V]``."""
@@ -166,8 +186,7 @@ def memory_step(q, k, v, z, zb, foff: int, cap: float, q_scale: float, bufs, rb,
         load_lin_ext().memory_step(q, k, v, z, zb, int(foff), float(cap), float(q_scale), S, bufs["keys"], bufs["peak"], rb.slots, rb.past, w, gate,
                                    float(eps), float(out_scale), y)
         return y
-    o = memory_scan(q, k, v, z, zb, foff, cap, q_scale, bufs, rb)
-    return gated_norm(o, gate, w, eps, GATE_NONE if gate is None else GATE_SIGMOID, y, S.shape[1], S.shape[3], per_head=True, out_scale=out_scale)
+    return memory_prompt(q, k, v, z, zb, foff, cap, q_scale, bufs, rb, w, gate, eps, y, out_scale)
 
 
 def gated_norm(o, gate, w, eps: float, act: int, y, H: int, V: int, *, per_head: bool, out_scale: float = 1.0):
