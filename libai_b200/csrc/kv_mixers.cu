@@ -1296,7 +1296,7 @@ int lbk_heads_prepare(void* q, long ldq, void* k, long ldk, const void* v, long 
   if (D > QK_MAXD || V > QK_MAXD || 2 * half > D || (base && !table && L < 1) || (table && (!base || page < 1))) return -1;
   const int unit0 = (qn || half) ? 0 : H, units = base ? H + 2 * G : H + G;
   if (unit0 >= units || (unit0 && !base)) return 0;
-  const int per = tokens * (units - unit0) <= 148 * 16 ? 1 : 8;
+  const int per = tokens * (units - unit0) <= 148 * 16 ? 1 : 12;
   const long warps = tokens * ((units - unit0 + per - 1) / per);
   const CacheRows cr{base, table, L, max_pages, page, G * (D + V), G * D};
   const int esz = dtype ? 2 : 4;

@@ -503,9 +503,9 @@ decay_scan_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, lo
 // maximum (0 at the start of a sequence) keeps the state in range,
 //   m_t = max(f + m_(t-1), i),   decay = exp(f + m_(t-1) - m_t),   write = exp(i - m_t),   floor = exp(-m_t),
 //   S <- decay S + write k v^T,   z <- decay z + write k,   o = S^T q / (max(|z q|, floor) + 1e-6).
-// memory_gates_kernel: one warp per (sequence, head) turns the logits of the step into gates [H][3][tokens] = decay, write, floor, 32 tokens
-// at a time: with F_t = sum of f over the group, m_t = max(F_t + m_in, max_s (i_s + F_t - F_s)) is a scan of (f, i) pairs under
-// (F1 + F2, max(M1 + F2, M2)).  mx [slots, H] holds the running maximum between steps.  `chunk` > 0 (a multiple of 32): gates
+// memory_gates_kernel: one block per (sequence, head) turns the logits of the step into gates [H][3][tokens] = decay, write, floor, groups of
+// 32 tokens side by side, a warp each: with F_t = sum of f over the group, m_t = max(F_t + m_in, max_s (i_s + F_t - F_s)) is a scan of (f, i) pairs under
+// (F1 + F2, max(M1 + F2, M2)).  mx [slots, H] holds the running maximum between steps.  `chunk` > 0 (a multiple of 32 that divides a turn's tokens): gates
 // [H][6][tokens] instead, for the chunked form (memory_mixers.cu): F from the chunk's start in two numbers (upper part and rest, so that
 // differences keep their digits), i, m, exp(F + m before the chunk - m), exp(-m).
 // ------------------------------------------------------------------------------------------------------------------
@@ -526,36 +526,50 @@ __device__ __forceinline__ void add_exact(float& h, float& l, float ph, float pl
   h = s;
 }
 
-__global__ void memory_gates_kernel(const float* __restrict__ z, long ldz, int foff, const float* __restrict__ zb, float cap,
-                                    float* __restrict__ mx, const int* __restrict__ seq_off, const int* __restrict__ slots,
-                                    const int* __restrict__ past, float* __restrict__ gates, long tokens, int B, int H, int chunk) {
-  const int wid = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (wid >= B * H) return;
-  const int b = wid / H, h = wid - b * H;
+constexpr int MG_WARPS = 8;            // groups of 32 tokens that a block scans side by side
+
+__global__ void __launch_bounds__(32 * MG_WARPS)
+memory_gates_kernel(const float* __restrict__ z, long ldz, int foff, const float* __restrict__ zb, float cap, float* __restrict__ mx,
+                    const int* __restrict__ seq_off, const int* __restrict__ slots, const int* __restrict__ past, float* __restrict__ gates,
+                    long tokens, int H, int chunk) {
+  __shared__ float gF[2][MG_WARPS], gFl[2][MG_WARPS], gM[2][MG_WARPS];   // a group's totals (two buffers: one barrier per turn)
+  const int b = blockIdx.x / H, h = blockIdx.x - b * H, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long tok0 = seq_off[b];
   const int n = seq_off[b + 1] - seq_off[b];
   float* mslot = mx + (long)slots[b] * H + h;
-  float m = past[b] > 0 ? *mslot : 0.f;
+  float m = past[b] > 0 ? *mslot : 0.f;           // the maximum before the turn's tokens
   const float bi = zb[h], bf = zb[foff + h];
   float* g0 = gates + (long)h * (chunk ? 6 : 3) * tokens + tok0;
-  float Ch = 0.f, Cl = 0.f, m0 = m;               // F of the chunk so far, m before the chunk
-  for (int t0 = 0; t0 < n; t0 += 32) {
-    const int t = t0 + lane;
+  const float* zr = z + tok0 * ldz;
+  float zi = 0.f, zf = 0.f;
+  if (threadIdx.x < n) { zi = zr[threadIdx.x * ldz + h]; zf = zr[threadIdx.x * ldz + foff + h]; }
+  int buf = 0;
+  for (int t0 = 0; t0 < n; t0 += 32 * MG_WARPS, buf ^= 1) {
+    const int t = t0 + (int)threadIdx.x, tn = t + 32 * MG_WARPS;
     float li = -INFINITY, lf = 0.f;               // beyond the end: the maximum stays
-    if (t < n) memory_log_gates(z[(tok0 + t) * ldz + h] + bi, z[(tok0 + t) * ldz + foff + h] + bf, cap, li, lf);
+    if (t < n) memory_log_gates(zi + bi, zf + bf, cap, li, lf);
+    if (tn < n) { zi = zr[(long)tn * ldz + h]; zf = zr[(long)tn * ldz + foff + h]; }     // the next turn's logits, in flight meanwhile
     float F = lf, Fl = 0.f, M = li;
 #pragma unroll
     for (int d = 1; d < 32; d <<= 1) {
       const float Fp = __shfl_up_sync(0xffffffffu, F, d), Flp = __shfl_up_sync(0xffffffffu, Fl, d), Mp = __shfl_up_sync(0xffffffffu, M, d);
       if (lane >= d) { M = fmaxf(Mp + F, M); add_exact(F, Fl, Fp, Flp); }
     }
-    const float mt = fmaxf(F + m, M);
-    float mp = __shfl_up_sync(0xffffffffu, mt, 1);
-    if (lane == 0) mp = m;
+    if (lane == 31) { gF[buf][warp] = F; gFl[buf][warp] = Fl; gM[buf][warp] = M; }
+    __syncthreads();
+    float run = m, mine = m, m0 = m;              // the maximum before this warp's group, and before its chunk
+#pragma unroll
+    for (int u = 0; u < MG_WARPS; ++u) {
+      if (u == warp) mine = run;
+      if (chunk && u <= warp && (u * 32) % chunk == 0) m0 = run;
+      run = fmaxf(gF[buf][u] + run, gM[buf][u]);
+    }
+    m = run;
+    const float mt = fmaxf(F + mine, M);
     if (chunk) {
-      if (t0 % chunk == 0) { Ch = Cl = 0.f; m0 = m; }
+      float Ch = 0.f, Cl = 0.f;                   // F of the chunk's groups before this one
+      for (int u = warp - (warp * 32 % chunk) / 32; u < warp; ++u) add_exact(Ch, Cl, gF[buf][u], gFl[buf][u]);
       add_exact(F, Fl, Ch, Cl);
-      Ch = __shfl_sync(0xffffffffu, F, 31); Cl = __shfl_sync(0xffffffffu, Fl, 31);
       if (t < n) {
         g0[t] = F;
         g0[tokens + t] = Fl;
@@ -564,14 +578,17 @@ __global__ void memory_gates_kernel(const float* __restrict__ z, long ldz, int f
         g0[4 * tokens + t] = expf((F + (m0 - mt)) + Fl);
         g0[5 * tokens + t] = expf(-mt);
       }
-    } else if (t < n) {
-      g0[t] = expf(lf + mp - mt);
-      g0[tokens + t] = expf(li - mt);
-      g0[2 * tokens + t] = expf(-mt);
+    } else {
+      float mp = __shfl_up_sync(0xffffffffu, mt, 1);
+      if (lane == 0) mp = mine;
+      if (t < n) {
+        g0[t] = expf(lf + mp - mt);
+        g0[tokens + t] = expf(li - mt);
+        g0[2 * tokens + t] = expf(-mt);
+      }
     }
-    m = __shfl_sync(0xffffffffu, mt, 31);
   }
-  if (lane == 0) *mslot = m;
+  if (threadIdx.x == 0) *mslot = m;
 }
 
 // One token per sequence: gates, state update, read-out, per-head RMS norm, weight w [H*V] and sigmoid gate in one block per (sequence, head).
@@ -832,8 +849,8 @@ int lbl_decay_scan(const void* q, long ldq, const void* k, long ldk, const void*
 int lbl_memory_gates(const float* z, long ldz, int foff, const float* zb, float cap, float* mx, const int* seq_off, const int* slots,
                      const int* past, float* gates, long tokens, int B, int H, int chunk, cudaStream_t s) {
   if (B == 0 || tokens == 0) return 0;
-  if (!(cap > 0.f) || chunk % 32) return -1;
-  memory_gates_kernel<<<(unsigned)(B * H), 32, 0, s>>>(z, ldz, foff, zb, cap, mx, seq_off, slots, past, gates, tokens, B, H, chunk);
+  if (!(cap > 0.f) || (chunk && (chunk % 32 || (32 * MG_WARPS) % chunk))) return -1;
+  memory_gates_kernel<<<(unsigned)(B * H), 32 * MG_WARPS, 0, s>>>(z, ldz, foff, zb, cap, mx, seq_off, slots, past, gates, tokens, H, chunk);
   LAUNCH_END();
 }
 

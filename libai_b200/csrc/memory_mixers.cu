@@ -47,7 +47,8 @@ __device__ __forceinline__ void split3(float x, float y, uint32_t (&p)[3]) {
     x -= t.x; y -= t.y;
   }
 }
-__device__ __forceinline__ float sigmoid1(float x) { return 1.f / (1.f + expf(-x)); }
+// the output gate's activation, rounded to bf16 with the result
+__device__ __forceinline__ float sigmoid1(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 
 template <int DB, int NB>              // DB: key channels / 16 (padded), NB: blocks of 8 value columns per warp
 struct McCfg {
@@ -289,18 +290,22 @@ memory_chunk_kernel(const bf16* __restrict__ q, long ldq, const bf16* __restrict
       }
       const uint32_t vrow = smem_u32(sV + (k2 * 16 + (lane & 15)) * VS + cw + (lane >> 4) * 8);
 #pragma unroll
-      for (int nb = 0; nb < NB; nb += 2) {
-        uint32_t bb[4];
-        ldsm_x4_trans(bb, vrow + nb * 16);
-        if (k2 <= wr) {
+      for (int nb = 0; nb < NB; nb += 4) {                              // products of one part go to four accumulators in turn
+        uint32_t ba[4], bb[4];
+        ldsm_x4_trans(ba, vrow + nb * 16);
+        ldsm_x4_trans(bb, vrow + nb * 16 + 32);
 #pragma unroll
-          for (int u = 0; u < 3; ++u) { mma_bf16(o[nb], pa[u], bb[0], bb[1]); mma_bf16(o[nb + 1], pa[u], bb[2], bb[3]); }
-        }
-        if (owner) {
+        for (int u = 0; u < 3; ++u) {
+          if (k2 <= wr) {
+            mma_bf16(o[nb], pa[u], ba[0], ba[1]); mma_bf16(o[nb + 1], pa[u], ba[2], ba[3]);
+            mma_bf16(o[nb + 2], pa[u], bb[0], bb[1]); mma_bf16(o[nb + 3], pa[u], bb[2], bb[3]);
+          }
+          if (owner) {
 #pragma unroll
-          for (int i = 0; i < MB; ++i) {
-#pragma unroll
-            for (int u = 0; u < 3; ++u) { mma_bf16(s[i][nb], ka[i][u], bb[0], bb[1]); mma_bf16(s[i][nb + 1], ka[i][u], bb[2], bb[3]); }
+            for (int i = 0; i < MB; ++i) {
+              mma_bf16(s[i][nb], ka[i][u], ba[0], ba[1]); mma_bf16(s[i][nb + 1], ka[i][u], ba[2], ba[3]);
+              mma_bf16(s[i][nb + 2], ka[i][u], bb[0], bb[1]); mma_bf16(s[i][nb + 3], ka[i][u], bb[2], bb[3]);
+            }
           }
         }
       }

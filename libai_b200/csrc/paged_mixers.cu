@@ -970,7 +970,7 @@ int lbp_sandwich_residual(float* x, const float* y, long ldy, const float* y2, l
                    al(bw2, 4 * esz) && al(pw, 4 * esz) && al(add, 4 * esz) && al(nw, 4 * esz) && al(h, 4 * esz);
 #define SRA(TT) x, y, ldy, y2, ldy2, (const TT*)bw1, (const TT*)bw2, bscale, (const TT*)pw, mult, (const TT*)add, (const TT*)nw, eps, (TT*)h, ldh, n
   if (vec && n / 4 <= 2048) {
-    const int quads = n / 4, items = quads <= 256 ? 1 : 2;
+    const int quads = n / 4, items = quads <= 64 ? 1 : 2;
     const int threads = (((quads + items - 1) / items + 31) / 32) * 32;
 #define SR(TT) { if (items == 1) sandwich_residual_vec_kernel<TT, 1><<<(unsigned)rows, threads, 0, s>>>(SRA(TT)); \
                  else sandwich_residual_vec_kernel<TT, 2><<<(unsigned)rows, threads, 0, s>>>(SRA(TT)); }

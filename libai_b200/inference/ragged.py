@@ -87,8 +87,8 @@ class RaggedBatch:
             self.offsets.append(self.offsets[-1] + n)
         self.tokens = self.offsets[-1]
         self.single = all(n == 1 for n in self.lens)          # every sequence goes on by one token
-        tok_seq = [b for b, n in enumerate(self.lens) for _ in range(n)]
-        packed = torch.tensor(self.offsets + self.slot_list + self.past_list + tok_seq, dtype=torch.int32)
+        tok_seq = torch.repeat_interleave(torch.arange(self.B, dtype=torch.int32), torch.tensor(self.lens))
+        packed = torch.cat([torch.tensor(self.offsets + self.slot_list + self.past_list, dtype=torch.int32), tok_seq])
         packed = packed.to(self.device, non_blocking=True)
         B = self.B
         self.seq_off, self.slots, self.past = packed[: B + 1], packed[B + 1: 2 * B + 1], packed[2 * B + 1: 3 * B + 1]

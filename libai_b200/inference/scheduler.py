@@ -9,6 +9,7 @@ logits processors / warpers (greedy when none samples).
 from __future__ import annotations
 
 import os
+from array import array
 from typing import Dict, Hashable, List, Optional, Sequence, Tuple
 
 import torch
@@ -83,10 +84,13 @@ class RequestScheduler:
             if logits is not None:
                 return logits if any(want for _, _, want in entries) else None
         rb = RaggedBatch(lens, slots, [self.cache.length[s] for s in slots], self.device)
-        flat = [t for _, toks, _ in entries for t in toks]
+        flat = array("q")
+        for _, toks, _ in entries:
+            flat.fromlist(toks) if isinstance(toks, list) else flat.extend(toks)
         rows = [rb.offsets[b] + w for b, (_, _, want) in enumerate(entries) for w in want]
-        packed = torch.tensor(flat + rows, dtype=torch.long).to(self.device, non_blocking=True)
-        tokens, row_idx = packed[: len(flat)], packed[len(flat):]
+        flat.extend(rows)
+        packed = torch.frombuffer(flat, dtype=torch.long).to(self.device, non_blocking=True)
+        tokens, row_idx = packed[: rb.tokens], packed[rb.tokens:]
         logits = self.model.step(tokens, rb, row_idx)
         return logits if rows else None
 
