@@ -997,7 +997,7 @@ def kernel_table_fogezen(s, batch, prompt):
     cache.prepare(slots, [prompt + 1] * batch)
     pages, state = cache.buffers(paged), cache.buffers(mem)
     pages["pool"].copy_(rnd(*pages["pool"].shape))
-    freq, nofreq = KF.rotary_frequencies(D, 2e4)[0].to(dev), torch.zeros(0, device=dev)
+    freq, nofreq = KF.rotary_frequencies(D, 1e4)[0].to(dev), torch.zeros(0, device=dev)
     half = KF.rotary_frequencies(D // 2, 1e6)[0].to(dev)
     w, wd = torch.zeros(n, dtype=bf, device=dev), torch.ones(D, dtype=bf, device=dev)
     wm, zb = torch.ones(H * D, dtype=bf, device=dev), torch.zeros(2 * H, device=dev)
