@@ -913,7 +913,7 @@ def fogezen_config(s):
     feed-forwards."""
     D, H = s["dim"], s["heads"]
     heads = {"heads": H, "kv_heads": s["kv_heads"], "dim": D, "vdim": D, "scale": D ** -0.5}
-    par = {"left": dict(heads, mask={"size": s["reach"]}, rot={"dims": D, "base": 20000.0}), "right": {"heads": H, "dim": D // 2, "vdim": D, "gate_cap": 15.0}}
+    par = {"left": dict(heads, mask={"size": s["reach"]}, rot={"dims": D, "base": 10000.0}), "right": {"heads": H, "dim": D // 2, "vdim": D, "gate_cap": 15.0}}
     att = dict(heads, q_temp={"coef": 0.1, "every": 512})
     mlp = {"kind": "dense", "ff": s["ff"]}
     layers = [{"type": "attention", "mixer": att, "mlp": mlp} if i % 2 else {"type": "parallel", "mixer": par, "mlp": mlp} for i in range(s["blocks"])]
